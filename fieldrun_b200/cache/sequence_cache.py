@@ -8,7 +8,7 @@ pages: a sequence holds ``ceil(length / 64)`` pages per group and a table maps
 (slot, position // 64) to a page.  Cache lines whose needs are the same (number
 of key/value heads, key and value head sizes, all keys, a window of them or chunks) form a *group* with
 a store, a page pool and a table of its own; a windowed group gives a page back
-as soon as every key on it lies outside the window, a chunked group as soon as the
+as soon as every key on it lies outside the window (pages that hold the first tokens of a line that keeps those stay), a chunked group as soon as the
 sequence has left the chunks that the page holds.  What is cached is K after
 norm and rotary and V as projected (src/minimax.rs:262-268).
 
@@ -42,12 +42,33 @@ class CacheNeed:
     state_shape: tuple[int, ...] = ()    # state per sequence; () for none
     state_dtype: str = "float32"         # "float32" | "bfloat16" | "int32"
     values_in_keys: bool = False         # a key's value is a part of its key row: the line has no value pages
+    value_heads: int = 0                 # value heads, where several key heads share one; 0: one for every key head
+    keep_first: int = 0                  # with a window: the sequence's first tokens stay visible beside it
 
     @property
     def group_key(self) -> tuple | None:
         if not self.kv_heads:
             return None
-        return (self.kv_heads, self.head_dim, self.window, 0 if self.values_in_keys else self.value_dim or self.head_dim, self.chunk)
+        return (self.kv_heads, self.head_dim, self.window, 0 if self.values_in_keys else self.value_dim or self.head_dim, self.chunk,
+                self.value_heads or self.kv_heads, self.keep_first if self.window is not None else 0)
+
+    @property
+    def copy_floats(self) -> int:
+        """Floats in one of the two copies of a state of shape (2, floats); 0 without a state."""
+        if not self.state_shape:
+            return 0
+        if len(self.state_shape) != 2 or self.state_shape[0] != 2 or self.state_dtype != "float32":
+            raise ValueError(f"a state of shape {self.state_shape} and type {self.state_dtype} has no place for another part's: "
+                             "that takes (2, floats) in float32")
+        return self.state_shape[1]
+
+    def with_state_behind(self, floats: int) -> "CacheNeed":
+        """This need with ``floats`` more floats in each copy of its state, behind what is there: one line then holds the
+        state of two parts."""
+        from dataclasses import replace
+        if floats <= 0:
+            return self
+        return replace(self, state_shape=(2, self.copy_floats + floats), state_dtype="float32")
 
     def shared_with(self, reader: "CacheNeed") -> "CacheNeed":
         """What a line needs that this need's run writes and a run with need ``reader`` reads as well: the two may
@@ -69,7 +90,7 @@ class LineView:
     """What a mixer sees of its cache line."""
 
     keys: torch.Tensor | None            # [num_pages, kv_heads, PAGE_TOKENS, head_dim]
-    values: torch.Tensor | None          # [num_pages, kv_heads, value_dim, PAGE_TOKENS]; value_dim 0: values lie in the keys
+    values: torch.Tensor | None          # [num_pages, value heads, value_dim, PAGE_TOKENS]; value_dim 0: values lie in the keys
     page_table: torch.Tensor | None      # int32 [num_slots, max_pages]; -1 where no page is held
     window: int | None
     state: torch.Tensor | None           # [num_slots, *state_shape] in the need's state_dtype
@@ -77,12 +98,14 @@ class LineView:
 
 class _Group:
     def __init__(self, key, lines, num_pages, num_slots, dtype, device, allocate):
-        self.kv_heads, self.head_dim, self.window, self.value_dim, self.chunk = key
+        self.kv_heads, self.head_dim, self.window, self.value_dim, self.chunk, self.value_heads, keep_first = key
+        self.keep_pages = pages_for(keep_first)                      # pages that a sequence keeps to its end
         self.lines = list(lines)
         self.num_pages = num_pages
         self.pool = IndexPool(num_pages, "page")
         self.table = np.full((num_slots, num_pages), -1, dtype=np.int32)
-        self.first_page = np.zeros(num_slots, dtype=np.int64)        # first page index still held
+        # first page index still held (behind the kept ones, which are held as long as the sequence is)
+        self.first_page = np.zeros(num_slots, dtype=np.int64)
         self.end_page = np.zeros(num_slots, dtype=np.int64)          # one past the last page held
         self.dirty: list[tuple[int, int, int]] = []
         self.fresh: list[int] = []           # pages given out since the last sync whose old contents may be read
@@ -91,7 +114,7 @@ class _Group:
             self.keys = torch.zeros(shape, dtype=dtype, device=device)
             # within a page the values lie transposed, [head_dim, PAGE_TOKENS]: the product P @ V then reads
             # runs of neighbouring keys
-            self.values = torch.zeros(shape[:3] + (self.value_dim, PAGE_TOKENS), dtype=dtype, device=device)
+            self.values = torch.zeros(shape[:2] + (self.value_heads, self.value_dim, PAGE_TOKENS), dtype=dtype, device=device)
             self.table_dev = torch.full((num_slots, num_pages), -1, dtype=torch.int32, device=device)
         else:
             self.keys = self.values = self.table_dev = None
@@ -123,7 +146,7 @@ class _Group:
         if self.chunk is not None:
             # ... and only keys of its own chunk, which begins at or after the chunk of position `length`
             first_needed = max(first_needed, (length // self.chunk * self.chunk) // PAGE_TOKENS)
-        lo = int(self.first_page[slot])
+        lo = max(int(self.first_page[slot]), self.keep_pages)
         hi = min(first_needed, int(self.end_page[slot]))
         if hi <= lo:
             return
@@ -134,12 +157,14 @@ class _Group:
         self.dirty.append((slot, lo, hi))
 
     def release_all(self, slot: int) -> None:
-        lo, hi = int(self.first_page[slot]), int(self.end_page[slot])
-        for index in range(lo, hi):
-            self.pool.free(int(self.table[slot, index]))
-            self.table[slot, index] = -1
-        if hi > lo:
-            self.dirty.append((slot, lo, hi))
+        first, end = int(self.first_page[slot]), int(self.end_page[slot])
+        kept = min(self.keep_pages, first)                 # pages before `first` that were never given back
+        for lo, hi in ((0, kept), (first, end)):
+            for index in range(lo, hi):
+                self.pool.free(int(self.table[slot, index]))
+                self.table[slot, index] = -1
+            if hi > lo:
+                self.dirty.append((slot, lo, hi))
         self.first_page[slot] = 0
         self.end_page[slot] = 0
 

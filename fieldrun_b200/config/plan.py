@@ -40,6 +40,8 @@ class LayerSpec:
     # norms behind the sublayers, for a block that has a norm on both sides of each (``sandwich_norm``)
     mixer_out_norm: Optional[PartSpec] = None
     feed_forward_out_norm: Optional[PartSpec] = None
+    # a part between the mixer's norm and the mixer (category ``mixer_input``), which may keep a state of its own
+    mixer_input: Optional[PartSpec] = None
 
 
 @dataclass(frozen=True)

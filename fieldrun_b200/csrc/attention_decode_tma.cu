@@ -1,5 +1,5 @@
-// One-token attention over the cache with the pages brought into shared memory by TMA (bfloat16, head
-// sizes 64 and 128).
+// One-token attention over the cache with the pages brought into shared memory by TMA (bfloat16, key heads of 64
+// and 128 entries, value heads of the same size or twice it up to 128).
 //
 // The formula is the reference's (src/minimax.rs:270-281).  A block takes a run of pages of one kv head of
 // one sequence: `chunks_per_block` chunks of 256 keys.  Three warps take the run's pages in turn (warp w the
@@ -8,7 +8,7 @@
 // results are combined through shared memory and written as one partial result, and the merge kernel adds
 // the blocks' partial results in order.
 //
-// A fourth warp asks for the pages: every page's keys [64][HD] and transposed values [HD][64] are copied by
+// A fourth warp asks for the pages: every page's keys [64][HD] and transposed values [VD][64] are copied by
 // cp.async.bulk.tensor into shared memory (128-byte swizzle).  Each warp has a stage for keys and a stage for
 // values of its own, each announced on an mbarrier and given back on another once the warp has multiplied
 // it; the next page's keys are on their way while the warp is at the present page's softmax and values.
@@ -44,7 +44,7 @@ struct DecodeTmaParams {
 
 // Warp w's page number n (the run's page 3 n + w) has its keys in stage 2 w and its values in stage 2 w + 1,
 // each on that stage's use n.
-template <int HD>
+template <int HD, int VD>
 __global__ void __launch_bounds__(DT_THREADS, 2)
 attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                             DecodeTmaParams params) {
@@ -53,8 +53,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     // go out before that kernel has ended; the warps that multiply wait for it before they read the queries.
     let_next_kernel_start();
     const DecodeAttnParams& p = params.a;
-    constexpr int STAGE_BYTES = FRB_PAGE * HD * 2;
-    constexpr int O_STRIDE = HD + 8;
+    constexpr int K_BYTES = FRB_PAGE * HD * 2, V_BYTES = FRB_PAGE * VD * 2, STAGE_BYTES = K_BYTES > V_BYTES ? K_BYTES : V_BYTES;
+    constexpr int O_STRIDE = VD + 8;
     static_assert(16 * O_STRIDE * 4 <= STAGE_BYTES, "a warp's partial result fits into a stage");
     extern __shared__ uint8_t dynamic[];
     __shared__ uint64_t full[DT_STAGES], empty[DT_STAGES];
@@ -68,11 +68,14 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     const int pos = p.seq_pos[b];
     const int slot = p.seq_slot[b];               // asked for together with the position: one wait, not two
     const int hi_key = pos, lo_key = first_visible_key(pos, p.window, p.chunk);
-    // the pages of this block that hold a key the token may see
+    // the pages of this block that hold a key the token may see: those of the first tokens that stay visible, then the window's
     const int pages_per_block = params.chunks_per_block * DT_CHUNK_PAGES;
-    const int first_page = max(part * pages_per_block, lo_key / FRB_PAGE);
-    const int end_page = min((part + 1) * pages_per_block, hi_key / FRB_PAGE + 1);
-    const int num_pages = end_page - first_page;
+    const int begin_page = part * pages_per_block, end_page = min((part + 1) * pages_per_block, hi_key / FRB_PAGE + 1);
+    const int first_page = max(begin_page, lo_key / FRB_PAGE);
+    const int kept = max(0, min(end_page, kept_runs(p.keep_first, FRB_PAGE, lo_key / FRB_PAGE)) - begin_page);
+    const int num_pages = kept + max(0, end_page - first_page);
+    auto page_of = [&](int n) { return n < kept ? begin_page + n : first_page + n - kept; };
+    const int vh = kvh / (p.num_kv_heads / p.v_heads);
     if (num_pages <= 0) return;                   // the merge skips these blocks
 
     if (threadIdx.x == 0) {
@@ -83,41 +86,40 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     __syncthreads();
 
     float row_max[2] = {-INFINITY, -INFINITY}, row_sum[2] = {0.f, 0.f};
-    float o[HD / 8][4];
+    float o[VD / 8][4];
 #pragma unroll
-    for (int n = 0; n < HD / 8; ++n)
+    for (int n = 0; n < VD / 8; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
     bool ok = true;
 
     if (warp == DT_WARPS) {
         if (lane == 0) {
-            const int* table = p.page_table + (size_t)slot * p.max_pages + first_page;
+            const int* table = p.page_table + (size_t)slot * p.max_pages;
             const int rounds = (num_pages + DT_WARPS - 1) / DT_WARPS;
-            const int newest = hi_key / FRB_PAGE - first_page;            // the page that the kernel before this one writes to
+            const int newest = kept + hi_key / FRB_PAGE - first_page;     // the page that the kernel before this one writes to
             bool waited = false;
             if (!params.early) { wait_for_previous_kernel(); waited = true; }
             for (int n = 0; n < rounds && ok; ++n) {
                 if (!waited && DT_WARPS * n + DT_WARPS > newest) { wait_for_previous_kernel(); waited = true; }
-                int rows[DT_WARPS];               // each page's first row in [pages * kv heads] rows of pages
+                int pages[DT_WARPS];
 #pragma unroll
-                for (int w = 0; w < DT_WARPS; ++w)
-                    rows[w] = DT_WARPS * n + w < num_pages ? table[DT_WARPS * n + w] * p.num_kv_heads + kvh : -1;
+                for (int w = 0; w < DT_WARPS; ++w) pages[w] = DT_WARPS * n + w < num_pages ? table[page_of(DT_WARPS * n + w)] : -1;
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {                 // the round's keys, then its values
 #pragma unroll
                     for (int w = 0; w < DT_WARPS; ++w) {
-                        if (rows[w] < 0 || !ok) continue;
+                        if (pages[w] < 0 || !ok) continue;
                         const int s = 2 * w + half;
                         if (n >= 1 && !bar_wait(&empty[s], (uint32_t)((n - 1) & 1), &failed)) { ok = false; continue; }
                         uint8_t* dst = stages + (size_t)s * STAGE_BYTES;
-                        bar_expect(&full[s], STAGE_BYTES);
+                        bar_expect(&full[s], half == 0 ? K_BYTES : V_BYTES);
                         if (half == 0) {
 #pragma unroll
                             for (int x = 0; x < HD / 64; ++x)
-                                load_2d(dst + (size_t)x * FRB_PAGE * 128, &map_k, 64 * x, rows[w] * FRB_PAGE, &full[s]);
+                                load_2d(dst + (size_t)x * FRB_PAGE * 128, &map_k, 64 * x, (pages[w] * p.num_kv_heads + kvh) * FRB_PAGE, &full[s]);
                         } else {
-                            load_2d(dst, &map_v, 0, rows[w] * HD, &full[s]);
+                            load_2d(dst, &map_v, 0, (pages[w] * p.v_heads + vh) * VD, &full[s]);
                         }
                     }
                 }
@@ -137,7 +139,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         float slope2[2];
         group_slopes(p.slopes, kvh * group, group, g, slope2);
         for (int n = 0; DT_WARPS * n + warp < num_pages && ok; ++n) {
-            const int key_base = (first_page + DT_WARPS * n + warp) * FRB_PAGE;
+            const int key_base = page_of(DT_WARPS * n + warp) * FRB_PAGE;
             const int k_stage = 2 * warp, v_stage = 2 * warp + 1;
             const uint32_t parity = (uint32_t)(n & 1);
             float s[8][4];
@@ -170,7 +172,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             }
             __syncwarp();
             if (lane == 0) bar_arrive(&empty[k_stage]);                  // this page's keys are no longer needed
-            // only a run's first and last page can hold keys the token may not see
+            // only the pages at the window's edge, behind the first tokens and of the token itself hold keys it may not see
             if (key_base < lo_key || key_base + FRB_PAGE - 1 > hi_key) {
 #pragma unroll
                 for (int m = 0; m < 2; ++m)
@@ -179,7 +181,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
 #pragma unroll
                         for (int e = 0; e < 4; ++e) {
                             const int key = key_base + 32 * m + 8 * t + 4 * (e & 1) + u;     // column 2 t + (e & 1)
-                            if (key < lo_key || key > hi_key) s[4 * m + u][e] = -INFINITY;
+                            if (!key_visible(key, lo_key, hi_key, p.keep_first)) s[4 * m + u][e] = -INFINITY;
                         }
             }
             float page_max[2] = {-INFINITY, -INFINITY};
@@ -203,7 +205,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             }
             if (__any_sync(0xffffffffu, grew)) {
 #pragma unroll
-                for (int n2 = 0; n2 < HD / 8; ++n2) {
+                for (int n2 = 0; n2 < VD / 8; ++n2) {
                     o[n2][0] *= corr[0]; o[n2][1] *= corr[0];
                     o[n2][2] *= corr[1]; o[n2][3] *= corr[1];
                 }
@@ -237,7 +239,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             {
                 const uint8_t* values = stages + (size_t)v_stage * STAGE_BYTES;
 #pragma unroll
-                for (int n2 = 0; n2 < HD / 8; ++n2) {
+                for (int n2 = 0; n2 < VD / 8; ++n2) {
                     // column g of this output tile is dimension 8 n2 + 4 (g & 1) + (g >> 1)
                     const int dim = 8 * n2 + 4 * (g & 1) + (g >> 1);
 #pragma unroll
@@ -267,7 +269,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     if (warp < DT_WARPS) {
         float* mine = reinterpret_cast<float*>(stages + (size_t)warp * STAGE_BYTES);
 #pragma unroll
-        for (int n2 = 0; n2 < HD / 8; ++n2) {                       // column 2 t + e is dimension 8 n2 + 4 e + t
+        for (int n2 = 0; n2 < VD / 8; ++n2) {                       // column 2 t + e is dimension 8 n2 + 4 e + t
             mine[g * O_STRIDE + 8 * n2 + t] = o[n2][0];
             mine[g * O_STRIDE + 8 * n2 + 4 + t] = o[n2][1];
             mine[(g + 8) * O_STRIDE + 8 * n2 + t] = o[n2][2];
@@ -279,8 +281,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         }
     }
     __syncthreads();
-    for (int idx = threadIdx.x; idx < group * HD; idx += DT_THREADS) {
-        const int r = idx / HD, d = idx - r * HD;
+    for (int idx = threadIdx.x; idx < group * VD; idx += DT_THREADS) {
+        const int r = idx / VD, d = idx - r * VD;
         float top = -INFINITY;
 #pragma unroll
         for (int w = 0; w < DT_WARPS; ++w) top = fmaxf(top, sm_m[w][r]);
@@ -294,29 +296,19 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             }
         }
         const size_t row = ((size_t)b * p.num_heads + (size_t)kvh * group + r) * p.max_chunks + part;
-        p.part_o[row * HD + d] = acc;
+        p.part_o[row * VD + d] = acc;
         if (d == 0) { p.part_ml[row * 2] = top; p.part_ml[row * 2 + 1] = sum; }
     }
 }
 
 // grid (head, sequence): merges the blocks' partial results of one (sequence, head), first block to last.
-template <int HD>
-__global__ void __launch_bounds__(HD) attention_decode_tma_merge_kernel(DecodeTmaParams params) {
+template <int VD>
+__global__ void __launch_bounds__(VD) attention_decode_tma_merge_kernel(DecodeTmaParams params) {
     after_previous_kernel();
-    const DecodeAttnParams& p = params.a;
-    const int head = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
-    const int pos = p.seq_pos[b];
-    const int lo_key = first_visible_key(pos, p.window, p.chunk);
-    const int keys_per_block = params.chunks_per_block * ATT_CHUNK;
-    // never beyond the partial results the launch has room for, whatever the position says
-    const int last = min(pos / keys_per_block, p.max_chunks - 1), first = min(lo_key / keys_per_block, last);
-    if (pos / keys_per_block >= p.max_chunks && d == 0) atomicExch(params.status, FRB_STATUS_TOO_LONG);   // keys were left out
-    const size_t row0 = ((size_t)b * p.num_heads + head) * p.max_chunks;
-    p.out[((size_t)b * p.num_heads + head) * HD + d] = __float2bfloat16_rn(merged_element<HD>(p.part_ml, p.part_o, row0, first, last, d,
-                                                                                                    p.sinks ? p.sinks[head] * 1.4426950408889634f : -INFINITY));
+    merge_head<VD>(params.a, params.chunks_per_block * ATT_CHUNK, params.status);
 }
 
-// As frb_attention_decode_mma, for head sizes 64 and 128.  num_pages: pages of the cache group (the tensor
+// As frb_attention_decode_mma, for key heads of 64 and 128.  num_pages: pages of the cache group (the tensor
 // maps cover all of them).  max_chunks: chunks of 256 keys of the longest sequence; part_o and part_ml need
 // room for ceil(max_chunks / chunks_per_block) partial results per (sequence, head).  chunks_per_block: chunks
 // that one block takes (at least 1).  status: one int on the device, zero before the call; 4 afterwards if a
@@ -325,41 +317,44 @@ FRB_API int frb_attention_decode_tma(const void* q, const void* k_pages, const v
                                      const int* page_table, int max_pages, const int* seq_pos, const int* seq_slot,
                                      float* part_o, float* part_ml, void* out, int num_seqs, int num_heads, int num_kv_heads,
                                      int head_dim, float scale, int window, int max_chunks, int chunks_per_block, int* status,
-                                     const float* slopes, int chunk, const float* sinks, float softcap, cudaStream_t stream) {
+                                     const float* slopes, int chunk, const float* sinks, float softcap, int v_dim, int keep_first,
+                                     int v_heads, const float* lam, float diff_eps, float diff_factor, cudaStream_t stream) {
     if (num_seqs == 0) return 0;
+    if (v_dim <= 0) v_dim = head_dim;
+    AttnExtras extras;
+    extras.slopes = slopes; extras.chunk = chunk; extras.sinks = sinks; extras.softcap = softcap; extras.v_dim = v_dim;
+    extras.keep_first = keep_first; extras.v_heads = v_heads; extras.lam = lam; extras.diff_eps = diff_eps; extras.diff_factor = diff_factor;
     const int group = num_kv_heads > 0 ? num_heads / num_kv_heads : 0;
     FRB_CHECK_ARG(num_kv_heads > 0 && num_heads % num_kv_heads == 0 && group <= 16,
                   "attention_decode_tma: %d heads over %d kv heads (groups of at most 16)", num_heads, num_kv_heads);
-    FRB_CHECK_ARG(head_dim == 64 || head_dim == 128, "attention_decode_tma: head_dim %d is neither 64 nor 128", head_dim);
+    FRB_CHECK_ARG((head_dim == 64 || head_dim == 128) && attention_sizes_built(head_dim, v_dim),
+                  "attention_decode_tma: head_dim %d with value heads of %d is not built", head_dim, v_dim);
     FRB_CHECK_ARG(num_seqs <= 65535 && num_kv_heads <= 65535, "attention_decode_tma: %d sequences exceed the grid", num_seqs);
     FRB_CHECK_ARG(chunks_per_block >= 1 && max_chunks >= 1, "attention_decode_tma: %d chunks per block", chunks_per_block);
-    CUtensorMap map_k, map_v;
-    const uint64_t kv_rows = (uint64_t)num_pages * num_kv_heads;
-    FRB_CHECK_ARG(map_rows_of_64(&map_k, k_pages, kv_rows * FRB_PAGE, head_dim, FRB_PAGE) &&
-                  map_rows_of_64(&map_v, v_pages, kv_rows * head_dim, FRB_PAGE, head_dim),
-                  "attention_decode_tma: cuTensorMapEncodeTiled failed or is not available");
     DecodeTmaParams params;
     DecodeAttnParams& p = params.a;
     const int parts = (max_chunks + chunks_per_block - 1) / chunks_per_block;
     p.q = (const bf16*)q; p.k_pages = (const bf16*)k_pages; p.v_pages = (const bf16*)v_pages; p.page_table = page_table;
     p.seq_pos = seq_pos; p.seq_slot = seq_slot; p.part_o = part_o; p.part_ml = part_ml; p.out = (bf16*)out;
     p.scale2 = scale * 1.4426950408889634f; p.window = window; p.max_pages = max_pages; p.num_heads = num_heads;
-    p.num_kv_heads = num_kv_heads; p.max_chunks = parts; p.status = status; p.slopes = slopes;
-    p.chunk = chunk; p.sinks = sinks;
-    p.cap_scale = softcap > 0.f ? scale / softcap : 0.f; p.cap2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+    p.num_kv_heads = num_kv_heads; p.max_chunks = parts; p.status = status;
+    if (fill_decode_extras("attention_decode_tma", p, head_dim, scale, extras)) return -1;
+    CUtensorMap map_k, map_v;
+    FRB_CHECK_ARG(map_rows_of_64(&map_k, k_pages, (uint64_t)num_pages * num_kv_heads * FRB_PAGE, head_dim, FRB_PAGE) &&
+                  map_rows_of_64(&map_v, v_pages, (uint64_t)num_pages * p.v_heads * v_dim, FRB_PAGE, v_dim),
+                  "attention_decode_tma: cuTensorMapEncodeTiled failed or is not available");
     params.chunks_per_block = chunks_per_block; params.status = status;
     static const int early = [] { const char* v = getenv("FIELDRUN_B200_ATTENTION_EARLY"); return !(v && v[0] == '0'); }();
     params.early = early;
-    dim3 grid(parts, num_kv_heads, num_seqs), merge_grid(num_heads, num_seqs);
-    const size_t smem = (size_t)DT_STAGES * FRB_PAGE * head_dim * 2 + 1024;
-    if (head_dim == 64) {
-        cudaFuncSetAttribute(attention_decode_tma_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        launch_dependent_resident(early ? 2 : 1, attention_decode_tma_kernel<64>, grid, dim3(DT_THREADS), smem, stream, map_k, map_v, params);
-        launch_dependent(attention_decode_tma_merge_kernel<64>, merge_grid, dim3(64), 0, stream, params);
-    } else {
-        cudaFuncSetAttribute(attention_decode_tma_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        launch_dependent_resident(early ? 2 : 1, attention_decode_tma_kernel<128>, grid, dim3(DT_THREADS), smem, stream, map_k, map_v, params);
-        launch_dependent(attention_decode_tma_merge_kernel<128>, merge_grid, dim3(128), 0, stream, params);
-    }
+    dim3 grid(parts, num_kv_heads, num_seqs), merge_grid(lam ? num_heads / 2 : num_heads, num_seqs);
+    const size_t smem = (size_t)DT_STAGES * FRB_PAGE * (head_dim > v_dim ? head_dim : v_dim) * 2 + 1024;
+#define FRB_LAUNCH_DECODE_TMA(HD, VD)                                                                                             \
+    cudaFuncSetAttribute(attention_decode_tma_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);            \
+    launch_dependent_resident(early ? 2 : 1, attention_decode_tma_kernel<HD, VD>, grid, dim3(DT_THREADS), smem, stream, map_k, map_v, params); \
+    launch_dependent(attention_decode_tma_merge_kernel<VD>, merge_grid, dim3(VD), 0, stream, params)
+    if (head_dim == 64 && v_dim == 64) { FRB_LAUNCH_DECODE_TMA(64, 64); }
+    else if (head_dim == 64) { FRB_LAUNCH_DECODE_TMA(64, 128); }
+    else { FRB_LAUNCH_DECODE_TMA(128, 128); }
+#undef FRB_LAUNCH_DECODE_TMA
     FRB_RETURN_LAUNCH("attention_decode_tma");
 }

@@ -12,7 +12,9 @@
 // sees only keys of its own chunk, floor(j / chunk) == floor(i / chunk), chunks counted from position 0), `sinks`
 // (a number per query head whose exponential joins the softmax's denominator, with no key and no value: it is not
 // scaled and counts once), `gate` (the head's output is multiplied by sigmoid(gate[t, h])) and `softcap` (the scaled
-// score s of every key becomes softcap * tanh(s / softcap) before anything else is done with it).
+// score s of every key becomes softcap * tanh(s / softcap) before anything else is done with it).  `keep_first`: beside the
+// window the query sees the sequence's first tokens.  Key heads in runs of num_kv_heads / num_v_heads share a value head (two
+// maps over one set of values); the output may be float32 whatever the operands are.
 #include "common.cuh"
 
 struct AttnParams {
@@ -27,6 +29,8 @@ struct AttnParams {
     const int* tok_pos;       // [T]
     const int* tok_slot;      // [T]
     void* out;                // [T, nh * vd]
+    int out_f32;              // the output is float32 whatever T is
+    int keep_first, v_heads;
     float scale;
     float softcap;            // > 0: the scaled score s becomes softcap * tanh(s / softcap); 0: none
     int window;               // 0: every earlier key
@@ -54,7 +58,9 @@ __global__ void attention_generic_kernel(AttnParams p) {
     const T* q = (const T*)p.q;
     const T* k_pages = (const T*)p.k_pages;
     const T* v_pages = (const T*)p.v_pages;
-    T* out = (T*)p.out;
+    const int vg = g / (p.num_kv_heads / p.v_heads);
+    const int first_block = lo / KEY_BLOCK, kept = kept_runs(p.keep_first, KEY_BLOCK, first_block);
+    const int blocks = kept + hi / KEY_BLOCK - first_block + 1;
 
     for (int hbase = 0; hbase < group; hbase += nwarps) {
         const int hl = hbase + warp;
@@ -68,26 +74,27 @@ __global__ void attention_generic_kernel(AttnParams p) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) acc[i] = 0.f;
 
-        for (int j0 = (lo / KEY_BLOCK) * KEY_BLOCK; j0 <= hi; j0 += KEY_BLOCK) {
+        for (int n = 0; n < blocks; ++n) {
+            const int j0 = run_at(n, kept, first_block) * KEY_BLOCK;
             __syncthreads();
             const int page = table[j0 / FRB_PAGE];
             const size_t head_base = ((size_t)page * p.num_kv_heads + g) * FRB_PAGE * hd;
-            const size_t value_base = ((size_t)page * p.num_kv_heads + g) * FRB_PAGE * vd;
+            const size_t value_base = ((size_t)page * p.v_heads + vg) * FRB_PAGE * vd;
             const int in_page = j0 % FRB_PAGE;
             for (int i = threadIdx.x; i < KEY_BLOCK * hd; i += blockDim.x) {
                 const int r = i / hd, d = i - r * hd;
-                const bool valid = (j0 + r >= lo) && (j0 + r <= hi);
+                const bool valid = key_visible(j0 + r, lo, hi, p.keep_first);
                 k_tile[r * (hd + 1) + d] = valid ? to_f32<T>(k_pages[head_base + (size_t)(in_page + r) * hd + d]) : 0.f;
             }
             for (int i = threadIdx.x; i < KEY_BLOCK * vd; i += blockDim.x) {
                 const int d = i / KEY_BLOCK, r = i - d * KEY_BLOCK;          // keys of one dim are neighbours in memory
-                const bool valid = (j0 + r >= lo) && (j0 + r <= hi);
+                const bool valid = key_visible(j0 + r, lo, hi, p.keep_first);
                 v_tile[r * vd + d] = valid ? to_f32<T>(v_pages[value_base + (size_t)d * FRB_PAGE + in_page + r]) : 0.f;
             }
             __syncthreads();
             if (active) {
                 const int j = j0 + lane;
-                const bool valid = (j >= lo) && (j <= hi);
+                const bool valid = key_visible(j, lo, hi, p.keep_first);
                 float s = 0.f;
                 const float* qr = q_rows + warp * hd;
                 const float* kr = k_tile + lane * (hd + 1);
@@ -126,7 +133,11 @@ __global__ void attention_generic_kernel(AttnParams p) {
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const int d = lane + 32 * i;
-                if (d < vd) out[((size_t)t * p.num_heads + head) * vd + d] = from_f32<T>(acc[i] * inv);
+                const size_t at = ((size_t)t * p.num_heads + head) * vd + d;
+                if (d < vd) {
+                    if (p.out_f32) ((float*)p.out)[at] = acc[i] * inv;
+                    else ((T*)p.out)[at] = from_f32<T>(acc[i] * inv);
+                }
             }
         }
     }
@@ -136,8 +147,12 @@ FRB_API int frb_attention_generic(const void* q, const void* k_pages, const void
                                   const int* page_table, int max_pages, const int* tok_pos, const int* tok_slot,
                                   void* out, int num_tokens, int num_heads, int num_kv_heads, int head_dim,
                                   float scale, int window, int v_dim, const float* slopes, int chunk, const float* sinks,
-                                  const float* gate, int gate_stride, float softcap, cudaStream_t stream) {
+                                  const float* gate, int gate_stride, float softcap, int keep_first, int num_v_heads, int out_f32,
+                                  cudaStream_t stream) {
     if (num_tokens == 0) return 0;
+    if (num_v_heads <= 0) num_v_heads = num_kv_heads;
+    FRB_CHECK_ARG(num_kv_heads % num_v_heads == 0, "attention: %d key heads over %d value heads", num_kv_heads, num_v_heads);
+    FRB_CHECK_ARG(keep_first >= 0 && !(keep_first > 0 && chunk > 0), "attention: %d first tokens together with chunks", keep_first);
     if (v_dim <= 0) v_dim = head_dim;
     FRB_CHECK_ARG(v_dim <= 256, "attention: v_dim %d is outside 1..256", v_dim);
     FRB_CHECK_ARG(head_dim >= 1 && head_dim <= 256, "attention: head_dim %d is outside 1..256", head_dim);
@@ -149,6 +164,7 @@ FRB_API int frb_attention_generic(const void* q, const void* k_pages, const void
     p.tok_slot = tok_slot; p.out = out; p.scale = scale; p.window = window; p.max_pages = max_pages;
     p.num_heads = num_heads; p.num_kv_heads = num_kv_heads; p.head_dim = head_dim; p.v_dim = v_dim; p.slopes = slopes;
     p.chunk = chunk; p.sinks = sinks; p.gate = gate; p.gate_stride = gate_stride; p.softcap = softcap;
+    p.keep_first = window > 0 ? keep_first : 0; p.v_heads = num_v_heads; p.out_f32 = out_f32;
     const int group = num_heads / num_kv_heads;
     const int nwarps = group < 8 ? group : 8;
     const size_t smem = ((size_t)KEY_BLOCK * (head_dim + 1) + (size_t)KEY_BLOCK * v_dim + (size_t)nwarps * head_dim) * sizeof(float);

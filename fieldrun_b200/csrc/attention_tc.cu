@@ -81,7 +81,8 @@ struct AttnTcParams {
     const int* seq_start;
     const int* seq_q_len;
     const int* cu_q_len;
-    bf16* out;                 // [T, nh * HD]
+    bf16* out;                 // [T, nh * VD]
+    float* out32;              // null, or the output in float32 instead
     int* status;
     float scale2;              // softmax scale * log2(e)
     int window, max_pages, num_heads, num_kv_heads;
@@ -89,13 +90,15 @@ struct AttnTcParams {
     int chunk;                 // 0, or a query sees only the keys of its own chunk of this many positions
     const float* sinks;        // null, or one number per query head whose exponential joins the softmax's denominator
     float cap_scale, cap2;     // CAPPED kernels (capped_score2): scale / cap and cap * log2(e)
+    int keep_first, v_heads;   // first tokens that stay visible beside the window; value heads (runs of key heads share one)
 };
 
 // grid (tile of 128 queries, head); the longest tiles of a sequence (its last ones) start first.
 // SLOPED: the scores carry a bias that falls with the distance between query and key (one more multiply-add on each
 // pair of scores; a page's maximum is then bounded from above by its largest score with the bias of its last key,
 // which is all the running maximum needs to be).
-template <int HD, bool SLOPED, bool CAPPED>
+// HD: size of a key head; VD: of a value head.
+template <int HD, int VD, bool SLOPED, bool CAPPED>
 __global__ void __launch_bounds__(AT_THREADS)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, AttnTcParams p) {
@@ -106,14 +109,14 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     __shared__ int failed_flag;
     volatile int* failed = &failed_flag;
     constexpr int KBLOCKS = HD / 64;                           // 64 dims = one 128-byte swizzled row
-    constexpr uint32_t Q_BYTES = AT_QUERIES * HD * 2, K_BYTES = FRB_PAGE * HD * 2, V_BYTES = HD * FRB_PAGE * 2;
+    constexpr uint32_t Q_BYTES = AT_QUERIES * HD * 2, K_BYTES = FRB_PAGE * HD * 2, V_BYTES = VD * FRB_PAGE * 2;
     constexpr uint32_t STAGE_BYTES = AT_STEP_PAGES * (K_BYTES + V_BYTES);
     constexpr uint32_t K_BLOCK_BYTES = AT_STEP_KEYS * 128;     // one 64-dim block of a step's keys: [128 keys][128 bytes]
     // Tensor memory: two buffers of 128 columns, each a step's S (a column per key; page h of the step in columns
     // 64 h ...) and then its P (two bfloat16 per column, page h in columns 64 h ... 64 h + 31); O_0 and O_1.
     constexpr uint32_t SP_COL0 = 0, O_COL0 = 2 * AT_STEP_KEYS;
     constexpr uint32_t TMEM_COLS = 512;
-    static_assert(O_COL0 + AT_STEP_PAGES * 128 <= TMEM_COLS && HD <= 128 && AT_STEP_PAGES == 2, "tensor memory layout");
+    static_assert(O_COL0 + AT_STEP_PAGES * 128 <= TMEM_COLS && HD <= 128 && VD <= 128 && AT_STEP_PAGES == 2, "tensor memory layout");
 
     // The step's tables are not the work of the kernel before this one (it writes queries, keys and values): they
     // are read, and barriers and tensor memory set up, while that kernel still runs.
@@ -126,12 +129,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int* table = p.page_table + (size_t)p.seq_slot[b] * p.max_pages;
     const int last_key = start + min(q0 + AT_QUERIES - 1, q_len - 1);
     const int first_key = first_visible_key(start + q0, p.window, p.chunk);
-    const int first_page = first_key / FRB_PAGE, num_pages = last_key / FRB_PAGE - first_page + 1;
+    // the pages of the first tokens that stay visible, then those from the window on
+    const int first_page = first_key / FRB_PAGE, kept = kept_runs(p.keep_first, FRB_PAGE, first_page);
+    const int num_pages = kept + last_key / FRB_PAGE - first_page + 1;
+    const int vh = kvh / (p.num_kv_heads / p.v_heads);
     const int num_steps = (num_pages + AT_STEP_PAGES - 1) / AT_STEP_PAGES;     // a step: two pages, the last one maybe one
 
     uint8_t* base = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     uint8_t* q_tile = base;                                    // KBLOCKS tiles [128 x 64]
-    uint8_t* stage0 = base + Q_BYTES;                          // per stage: K (KBLOCKS tiles [128 keys x 64]) then V^T ([HD x 64] per page)
+    uint8_t* stage0 = base + Q_BYTES;                          // per stage: K (KBLOCKS tiles [128 keys x 64]) then V^T ([VD x 64] per page)
 
     if (threadIdx.x == 0) {
         bar_init(&q_full, 1);
@@ -165,22 +171,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 uint8_t* dst = stage0 + (size_t)s * STAGE_BYTES;
                 bar_expect(&kv_full[s], pages * (K_BYTES + V_BYTES));
                 for (int h = 0; h < pages; ++h) {
-                    const int page = table[first_page + AT_STEP_PAGES * j + h];
+                    const int page = table[run_at(AT_STEP_PAGES * j + h, kept, first_page)];
                     const int row = page * p.num_kv_heads + kvh;
 #pragma unroll
                     for (int kb = 0; kb < KBLOCKS; ++kb)
                         load_2d(dst + kb * K_BLOCK_BYTES + h * (FRB_PAGE * 128), &map_k, kb * 64, row * FRB_PAGE, &kv_full[s]);
-                    load_2d(dst + AT_STEP_PAGES * K_BYTES + h * V_BYTES, &map_v, 0, row * HD, &kv_full[s]);
+                    load_2d(dst + AT_STEP_PAGES * K_BYTES + h * V_BYTES, &map_v, 0, (page * p.v_heads + vh) * VD, &kv_full[s]);
                 }
             }
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            // float32 accumulate, bf16 operands, K-major; S: M 128 x N 128 (64 for a step of one page); O_h: M 128 x N HD.
+            // float32 accumulate, bf16 operands, K-major; S: M 128 x N 128 (64 for a step of one page); O_h: M 128 x N VD.
             // The MMAs of this thread run in the order of their issue.  So S of step j + 2 may be asked for into the
             // buffer of step j without a wait: P V of step j, which reads that buffer, was issued before, and was issued
             // only when the softmax of step j had read its S and written its P.
-            const uint32_t idesc_o = instr_desc_bf16(AT_QUERIES, HD);
+            const uint32_t idesc_o = instr_desc_bf16(AT_QUERIES, VD);
             const uint64_t q_desc = tile_desc(smem_addr(q_tile));
             bool ok = bar_wait(&q_full, 0, failed);
             if (!ok) atomicExch(p.status, 12);
@@ -240,7 +246,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (!bar_wait(&s_full[j & 1], (j >> 1) & 1, failed)) { if (ok && lane == 0) atomicExch(p.status, 16); ok = false; }
             fence_after_sync();
             const uint32_t mine = lane_base + SP_COL0 + AT_STEP_KEYS * (j & 1) + FRB_PAGE * half;
-            const int key0 = (first_page + AT_STEP_PAGES * j + half) * FRB_PAGE;
+            const int key0 = run_at(AT_STEP_PAGES * j + half, kept, first_page) * FRB_PAGE;
             uint32_t raw[FRB_PAGE / 16][16];
 #pragma unroll
             for (int c = 0; c < FRB_PAGE / 16; ++c) tmem_ld16(mine + 16 * c, raw[c]);
@@ -256,7 +262,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             }
             // Most pages lie wholly before the tile's first query (and inside the window): no key of theirs is
             // masked for any row of this warp, and the per-key comparisons are left out.
-            const bool open_page = __all_sync(0xffffffffu, valid && key0 + FRB_PAGE - 1 <= hi && key0 >= lo);
+            const bool open_page = __all_sync(0xffffffffu, valid && key0 + FRB_PAGE - 1 <= hi && (key0 >= lo || key0 + FRB_PAGE <= p.keep_first));
             const float bias0 = SLOPED ? slope2 * (float)(key0 - hi) : 0.f;      // the bias of the page's first key for this row
             float step_max;
             if (open_page) {
@@ -275,7 +281,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
                         const int key = key0 + 16 * c + i;
-                        const float v = key >= lo && key <= hi ? __uint_as_float(raw[c][i]) : -INFINITY;
+                        const float v = key_visible(key, lo, hi, p.keep_first) ? __uint_as_float(raw[c][i]) : -INFINITY;
                         raw[c][i] = __float_as_uint(v);
                         step_max = fmaxf(step_max, SLOPED ? fmaf(v, scale2, bias0 + slope2 * (float)(16 * c + i)) : v * scale2);
                     }
@@ -311,7 +317,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (!bar_wait(&kv_empty[(j - 1) % AT_STAGES], ((j - 1) / AT_STAGES) & 1, failed)) { if (ok && lane == 0) atomicExch(p.status, 18); ok = false; }
                 fence_after_sync();
 #pragma unroll 1
-                for (int c = 0; c < HD / 16; ++c) {
+                for (int c = 0; c < VD / 16; ++c) {
                     uint32_t o[16];
                     tmem_ld16(o_mine + 16 * c, o);
                     tmem_wait_ld();
@@ -354,8 +360,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // O_1 holds nothing if every step had one page (a sequence of at most 64 keys in reach)
         const float w0 = (half == 0 ? a_mine : a_other) * inv, w1 = num_pages > 1 ? (half == 0 ? a_other : a_mine) * inv : 0.f;
         if (ok && !*failed) {
-            constexpr int MINE = HD / 2;                       // output columns of this thread: [MINE half, MINE half + MINE)
-            bf16* dst = p.out + ((size_t)(tok0 + row) * p.num_heads + head) * HD + MINE * half;
+            constexpr int MINE = VD / 2;                       // output columns of this thread: [MINE half, MINE half + MINE)
+            const size_t at = ((size_t)(tok0 + row) * p.num_heads + head) * VD + MINE * half;
+            bf16* dst = p.out + at;
 #pragma unroll 1
             for (int c = 0; c < MINE / 16; ++c) {
                 uint32_t o0[16], o1[16];
@@ -368,6 +375,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     for (int i = 0; i < 16; ++i) {
                         y[i] = __uint_as_float(o0[i]) * w0;
                         if (num_pages > 1) y[i] = fmaf(__uint_as_float(o1[i]), w1, y[i]);
+                    }
+                    if (p.out32) {
+                        float4* dst32 = reinterpret_cast<float4*>(p.out32 + at + 16 * c);
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) dst32[i] = make_float4(y[4 * i], y[4 * i + 1], y[4 * i + 2], y[4 * i + 3]);
+                        continue;
                     }
                     uint4 lo4, hi4;
                     lo4.x = pack_bf16x2(y[0], y[1]);   lo4.y = pack_bf16x2(y[2], y[3]);
@@ -394,45 +407,56 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 
 // ----------------------------------------------------------------------------- host side
 
-// q bf16 [num_tokens, nh, hd]; k_pages [pages, nkv, 64, hd]; v_pages [pages, nkv, hd, 64]; tiles of 128 queries.
+// q bf16 [num_tokens, nh, hd]; k_pages [pages, nkv, 64, hd]; v_pages [pages, v_heads, vd, 64]; tiles of 128 queries.
 // status: one int on the device, zero before the call.
 FRB_API int frb_attention_prefill_tc(const void* q, int num_tokens, const void* k_pages, const void* v_pages, int num_pages,
                                      const int* page_table, int max_pages, const int* tile_seq, const int* tile_q0,
                                      int num_tiles, const int* seq_slot, const int* seq_start, const int* seq_q_len,
                                      const int* cu_q_len, void* out, int num_heads, int num_kv_heads, int head_dim, float scale,
                                      int window, int* status, const float* slopes, int chunk, const float* sinks,
-                                     float softcap, cudaStream_t stream) {
+                                     float softcap, int v_dim, int keep_first, int v_heads, int out_f32, cudaStream_t stream) {
     if (num_tiles == 0) return 0;
-    FRB_CHECK_ARG(head_dim == 64 || head_dim == 128, "tensor-core attention: head_dim %d is neither 64 nor 128", head_dim);
+    if (v_dim <= 0) v_dim = head_dim;
+    if (v_heads <= 0) v_heads = num_kv_heads;
+    FRB_CHECK_ARG((head_dim == 64 && (v_dim == 64 || v_dim == 128)) || (head_dim == 128 && v_dim == 128),
+                  "tensor-core attention: head_dim %d with value heads of %d is not built", head_dim, v_dim);
+    FRB_CHECK_ARG(num_kv_heads > 0 && num_kv_heads % v_heads == 0, "tensor-core attention: %d key heads over %d value heads", num_kv_heads, v_heads);
+    FRB_CHECK_ARG(keep_first >= 0 && !(keep_first > 0 && chunk > 0), "tensor-core attention: %d first tokens together with chunks", keep_first);
     FRB_CHECK_ARG(scale > 0.f, "tensor-core attention: a softmax scale of %g is not positive", (double)scale);
     FRB_CHECK_ARG(num_kv_heads > 0 && num_heads % num_kv_heads == 0 && num_heads <= 65535, "tensor-core attention: %d heads over %d kv heads",
                   num_heads, num_kv_heads);
     CUtensorMap map_q, map_k, map_v;
-    const uint64_t kv_rows = (uint64_t)num_pages * num_kv_heads;
     FRB_CHECK_ARG(map_rows_of_64(&map_q, q, num_tokens, (uint64_t)num_heads * head_dim, AT_QUERIES) &&
-                  map_rows_of_64(&map_k, k_pages, kv_rows * FRB_PAGE, head_dim, FRB_PAGE) &&
-                  map_rows_of_64(&map_v, v_pages, kv_rows * head_dim, FRB_PAGE, head_dim),
+                  map_rows_of_64(&map_k, k_pages, (uint64_t)num_pages * num_kv_heads * FRB_PAGE, head_dim, FRB_PAGE) &&
+                  map_rows_of_64(&map_v, v_pages, (uint64_t)num_pages * v_heads * v_dim, FRB_PAGE, v_dim),
                   "tensor-core attention: cuTensorMapEncodeTiled failed or is not available");
     AttnTcParams p;
     p.page_table = page_table; p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.seq_slot = seq_slot; p.seq_start = seq_start;
     p.seq_q_len = seq_q_len; p.cu_q_len = cu_q_len; p.out = (bf16*)out; p.status = status;
+    p.out32 = out_f32 ? (float*)out : nullptr; p.keep_first = window > 0 ? keep_first : 0; p.v_heads = v_heads;
     p.scale2 = scale * 1.4426950408889634f; p.window = window; p.max_pages = max_pages; p.num_heads = num_heads;
     p.num_kv_heads = num_kv_heads; p.slopes = slopes;
     p.chunk = chunk; p.sinks = sinks;
     p.cap_scale = softcap > 0.f ? scale / softcap : 0.f; p.cap2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     FRB_CHECK_ARG(!(softcap > 0.f && slopes), "tensor-core attention: capped scores together with distance slopes are not built");
-    const size_t smem = (size_t)AT_QUERIES * head_dim * 2 + (size_t)AT_STAGES * AT_STEP_PAGES * 2 * FRB_PAGE * head_dim * 2 + 1024;
+    const size_t smem = (size_t)AT_QUERIES * head_dim * 2 + (size_t)AT_STAGES * AT_STEP_PAGES * FRB_PAGE * (head_dim + v_dim) * 2 + 1024;
     dim3 grid(num_tiles, num_heads);
-#define FRB_LAUNCH_TC(HD, SLOPED, CAPPED)                                                                                    \
+#define FRB_LAUNCH_TC(HD, VD, SLOPED, CAPPED)                                                                                \
     do {                                                                                                                     \
-        cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, SLOPED, CAPPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        launch_dependent(attention_prefill_tc_kernel<HD, SLOPED, CAPPED>, grid, dim3(AT_THREADS), smem, stream, map_q, map_k, map_v, p); \
+        auto kernel = attention_prefill_tc_kernel<HD, VD, SLOPED, CAPPED>;                                                   \
+        cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                                \
+        launch_dependent(kernel, grid, dim3(AT_THREADS), smem, stream, map_q, map_k, map_v, p);                              \
     } while (0)
-    if (head_dim == 128) {
-        if (slopes) FRB_LAUNCH_TC(128, true, false); else if (softcap > 0.f) FRB_LAUNCH_TC(128, false, true); else FRB_LAUNCH_TC(128, false, false);
-    } else {
-        if (slopes) FRB_LAUNCH_TC(64, true, false); else if (softcap > 0.f) FRB_LAUNCH_TC(64, false, true); else FRB_LAUNCH_TC(64, false, false);
-    }
+#define FRB_LAUNCH_TC_SIZES(HD, VD)                                                                                          \
+    do {                                                                                                                     \
+        if (slopes) FRB_LAUNCH_TC(HD, VD, true, false);                                                                      \
+        else if (softcap > 0.f) FRB_LAUNCH_TC(HD, VD, false, true);                                                          \
+        else FRB_LAUNCH_TC(HD, VD, false, false);                                                                            \
+    } while (0)
+    if (head_dim == 128) FRB_LAUNCH_TC_SIZES(128, 128);
+    else if (v_dim == 128) FRB_LAUNCH_TC_SIZES(64, 128);
+    else FRB_LAUNCH_TC_SIZES(64, 64);
+#undef FRB_LAUNCH_TC_SIZES
 #undef FRB_LAUNCH_TC
     FRB_RETURN_LAUNCH("attention_prefill_tc");
 }

@@ -103,6 +103,16 @@ __device__ __forceinline__ int first_visible_key(int pos, int window, int chunk)
     return lo;
 }
 
+// A query whose sequence keeps its first `keep_first` tokens visible beside the window looks at two runs of pages: the
+// pages of those tokens, as far as they lie before `first_page`, then the pages from `first_page` on.  kept_runs() is the
+// number of units (pages, or any other size) of the first run, run_at() the unit that comes n-th; key_visible() what holds
+// inside them.
+__device__ __forceinline__ int kept_runs(int keep_first, int unit, int first) { return min((keep_first + unit - 1) / unit, first); }
+__device__ __forceinline__ int run_at(int n, int kept, int first) { return n < kept ? n : first + n - kept; }
+__device__ __forceinline__ bool key_visible(int key, int lo, int hi, int keep_first) {
+    return (key >= lo || key < keep_first) && key <= hi;
+}
+
 // A capped attention score for kernels that keep scores as powers of two: raw * scale becomes cap * tanh(raw * scale / cap),
 // returned times log2(e).  cap_scale = scale / cap, cap2 = cap * log2(e).  tanh(x) = 1 - 2 / (exp(2x) + 1) with the
 // hardware's exponential and reciprocal (errors of a few 1e-7 of the cap: these kernels round the weights to bfloat16).

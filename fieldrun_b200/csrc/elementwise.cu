@@ -217,8 +217,8 @@ FRB_API int frb_rmsnorm(float* x, const float* delta, const float* expert_y, con
 // ----------------------------------------------------------------------------- Q/K norm + rotary + cache write
 
 struct QkvParams {
-    const void* qkv;          // [T, (nh + nkv) * hd + nkv * vd], InT
-    const float* bias;        // [(nh + nkv) * hd + nkv * vd] added to the row before anything else, or null
+    const void* qkv;          // [T, (nh + nkv) * hd + nvh * vd], InT
+    const float* bias;        // [(nh + nkv) * hd + nvh * vd] added to the row before anything else, or null
     const void* q_weight;     // [nh*hd] or null: no norm
     const void* k_weight;     // [nkv*hd] or null
     const float* cos_table;   // [positions, rotary_dim/2]
@@ -228,7 +228,7 @@ struct QkvParams {
     const int* page_table;    // [slots, max_pages]
     void* q_out;              // [T, nh, hd] OutT
     void* k_pages;            // [pages, nkv, PAGE, hd] OutT
-    void* v_pages;            // [pages, nkv, hd, PAGE] OutT: values lie transposed within a page
+    void* v_pages;            // [pages, nvh, vd, PAGE] OutT: values lie transposed within a page
     float eps;
     int num_heads, num_kv_heads, head_dim, rotary_dim, interleaved, max_pages, write_cache, table_positions;
     int num_tokens, v_tiles;  // v_tiles: the grid's first v_tiles blocks write the values, 64 tokens of one kv head each
@@ -236,6 +236,7 @@ struct QkvParams {
     int tables_final;         // positions, slots and page table were complete before the kernel before this one began
     unsigned head_dim_inverse;   // ceil(2^32 / head_dim): the high word of n times this is n / head_dim for n < 2^24
     int v_dim;                // size of a value head (the keys' head_dim unless the design says otherwise)
+    int num_v_heads;          // value heads (the number of key heads unless several of those share one)
     unsigned v_dim_inverse;
     float q_temp_coef;        // the query is multiplied by 1 + coef * ln(floor((pos + 1) / every) + 1); 0: no such factor
     int q_temp_every;
@@ -259,7 +260,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_kernel(QkvParams p) {
     const int t = blockIdx.x;
     const int hd = p.head_dim;
     const int q_width = p.num_heads * hd, k_width = p.num_kv_heads * hd;
-    const int vd = p.v_dim, v_width = p.num_kv_heads * vd;
+    const int vd = p.v_dim, v_width = p.num_v_heads * vd;
     const int qk_width = q_width + k_width, all_width = qk_width + v_width;
     const int half = p.rotary_dim / 2;
     float* s_cos = raw + all_width;
@@ -345,7 +346,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_kernel(QkvParams p) {
         const float* vrow = raw + qk_width;
         for (int i = threadIdx.x; i < v_width; i += NORM_BLOCK) {
             const int head = i / vd, dim = i - head * vd;
-            const size_t at = (((size_t)page * p.num_kv_heads + head) * vd + dim) * FRB_PAGE + in_page;
+            const size_t at = (((size_t)page * p.num_v_heads + head) * vd + dim) * FRB_PAGE + in_page;
             ((OutT*)p.v_pages)[at] = from_f32<OutT>(vrow[i]);
         }
     }
@@ -363,7 +364,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_vec_kernel(QkvParams p
     __shared__ float scratch[64];
     const int hd = p.head_dim;
     const int q_width = p.num_heads * hd, k_width = p.num_kv_heads * hd;
-    const int vd = p.v_dim, v_width = p.num_kv_heads * vd;
+    const int vd = p.v_dim, v_width = p.num_v_heads * vd;
     const int qk_width = q_width + k_width, all_width = qk_width + v_width;
     int pos_early = 0, slot_early = 0, page_early = -1;
     // the blocks that transpose values come first in the grid: they run longest, and at the grid's end they ran alone
@@ -388,7 +389,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_vec_kernel(QkvParams p
         __shared__ int s_page[QKV_V_TOKENS], s_place[QKV_V_TOKENS];
         OutT* tile = reinterpret_cast<OutT*>(raw);                       // [vd][QKV_V_TOKENS + 2]
         const int index = blockIdx.x;
-        const int h = index % p.num_kv_heads, t0 = (index / p.num_kv_heads) * QKV_V_TOKENS;
+        const int h = index % p.num_v_heads, t0 = (index / p.num_v_heads) * QKV_V_TOKENS;
         const int count = min(QKV_V_TOKENS, p.num_tokens - t0);
         for (int j = threadIdx.x; j < count; j += NORM_BLOCK) {
             const int pos = p.tok_pos[t0 + j];
@@ -406,7 +407,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_vec_kernel(QkvParams p
         __syncthreads();
         for (int d = warp; d < vd; d += NORM_BLOCK / 32) {
             for (int j = lane; j < count; j += 32) {
-                const size_t at = (((size_t)s_page[j] * p.num_kv_heads + h) * vd + d) * FRB_PAGE + s_place[j];
+                const size_t at = (((size_t)s_page[j] * p.num_v_heads + h) * vd + d) * FRB_PAGE + s_place[j];
                 ((OutT*)p.v_pages)[at] = tile[d * (QKV_V_TOKENS + 2) + j];
             }
         }
@@ -501,7 +502,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_vec_kernel(QkvParams p
         const float* vrow = raw + qk_width;
         for (int i = threadIdx.x; i < v_width; i += NORM_BLOCK) {
             const int head = (int)__umulhi((unsigned)i, p.v_dim_inverse), dim = i - head * vd;
-            const size_t at = (((size_t)page * p.num_kv_heads + head) * vd + dim) * FRB_PAGE + in_page;
+            const size_t at = (((size_t)page * p.num_v_heads + head) * vd + dim) * FRB_PAGE + in_page;
             ((OutT*)p.v_pages)[at] = from_f32<OutT>(vrow[i]);
         }
     }
@@ -513,9 +514,12 @@ FRB_API int frb_qkv_prepare(const void* qkv, int in_dtype, const void* q_weight,
                             void* q_out, void* k_pages, void* v_pages, int out_dtype, int num_tokens, int num_heads,
                             int num_kv_heads, int head_dim, int rotary_dim, int interleaved, int write_cache,
                             int per_head, int tables_final, const float* bias, int v_dim, float q_temp_coef,
-                            int q_temp_every, cudaStream_t stream) {
+                            int q_temp_every, int num_v_heads, cudaStream_t stream) {
     if (num_tokens == 0) return 0;
     if (v_dim <= 0) v_dim = head_dim;
+    if (num_v_heads < 0) num_v_heads = num_kv_heads;
+    FRB_CHECK_ARG(num_v_heads == num_kv_heads || (num_v_heads > 0 && num_kv_heads % num_v_heads == 0),
+                  "qkv_prepare: %d key heads over %d value heads", num_kv_heads, num_v_heads);
     FRB_CHECK_ARG(q_temp_coef == 0.f || q_temp_every >= 1, "qkv_prepare: a query temperature every %d positions", q_temp_every);
     FRB_CHECK_ARG(rotary_dim % 2 == 0 && rotary_dim <= head_dim, "qkv_prepare: rotary_dim %d must be even and <= head_dim %d",
                   rotary_dim, head_dim);
@@ -529,9 +533,9 @@ FRB_API int frb_qkv_prepare(const void* qkv, int in_dtype, const void* q_weight,
     p.num_tokens = num_tokens; p.v_tiles = 0; p.per_head = per_head && (q_weight || k_weight);
     p.tables_final = tables_final;
     p.head_dim_inverse = (unsigned)((0x100000000ull + (unsigned)head_dim - 1) / (unsigned)head_dim);
-    p.bias = bias; p.v_dim = v_dim; p.q_temp_coef = q_temp_coef; p.q_temp_every = q_temp_every > 0 ? q_temp_every : 1;
+    p.bias = bias; p.v_dim = v_dim; p.num_v_heads = num_v_heads; p.q_temp_coef = q_temp_coef; p.q_temp_every = q_temp_every > 0 ? q_temp_every : 1;
     p.v_dim_inverse = (unsigned)((0x100000000ull + (unsigned)v_dim - 1) / (unsigned)v_dim);
-    const long long all_width = (long long)(num_heads + num_kv_heads) * head_dim + (long long)num_kv_heads * v_dim;
+    const long long all_width = (long long)(num_heads + num_kv_heads) * head_dim + (long long)num_v_heads * v_dim;
     FRB_CHECK_ARG(all_width < (1 << 24), "qkv_prepare: %d heads of %d", num_heads, head_dim);
     // per-head statistics: the squares of the q and k rows and one factor per head beside the rows
     const size_t smem = ((size_t)all_width + rotary_dim +
@@ -557,7 +561,7 @@ FRB_API int frb_qkv_prepare(const void* qkv, int in_dtype, const void* q_weight,
             const size_t bytes = smem > tile_bytes ? smem : tile_bytes;
             auto kernel = qkv_prepare_vec_kernel<InT, OutT, WT, 256>;
             if (bytes > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
-            const int v_blocks = (num_tokens + QKV_V_TOKENS - 1) / QKV_V_TOKENS * num_kv_heads;
+            const int v_blocks = (num_tokens + QKV_V_TOKENS - 1) / QKV_V_TOKENS * num_v_heads;
             p.v_tiles = v_blocks;
             launch_dependent(kernel, dim3(num_tokens + v_blocks), dim3(256), bytes, stream, p);
         } else {

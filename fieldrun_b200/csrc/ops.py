@@ -22,10 +22,10 @@ _P, _I, _F, _L = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlon
 _SIGNATURES = {
     "frb_embed_rows": "ppipiiifpi",
     "frb_rmsnorm": "pppppippifiipipi",
-    "frb_qkv_prepare": "pippifppipppipppiiiiiiiiiipifi",
+    "frb_qkv_prepare": "pippifppipppipppiiiiiiiiiipifii",
     "frb_wait_probe": "lpp",
     "frb_add_rows": "ppl",
-    "frb_attention_generic": "pppipipppiiiifiipippif",
+    "frb_attention_generic": "pppipipppiiiifiipippif" "iii",
     "frb_layernorm": "ppppfppiii",
     "frb_unary_unit": "ppili",
     "frb_softcap": "plf",
@@ -52,9 +52,9 @@ _SIGNATURES = {
     "frb_weighted_pair": "ppplff",
     "frb_sandwich_norm": "pppffpppippfpfiipipi",
     "frb_gated_delta_rule": "piiii" "piiii" "ppp" "ppp" "pll" "pi" "pii" "iiiii" "f",
-    "frb_attention_decode_mma": "ppppipppppiiiifiippipf",
-    "frb_attention_prefill_mma": "ppppippipppppiiifipipf",
-    "frb_attention_decode_tma": "pppipipppppiiiifiiippipf",
+    "frb_attention_decode_mma": "ppppipppppiiiifiippipf" "iiipff",
+    "frb_attention_prefill_mma": "ppppippipppppiiifipipf" "iiii",
+    "frb_attention_decode_tma": "pppipipppppiiiifiiippipf" "iiipff",
     "frb_expert_gemm_mma": "pppppppiipiiiiif",
     "frb_weight_stream": "pippppppiipiiiiiiipf",
     "frb_route_plan_small": "ppiiiifipppppppp",
@@ -62,7 +62,12 @@ _SIGNATURES = {
     "frb_router_logits": "ppiiip",
     "frb_expert_gemm_tc": "pipippppiipiiipif",
     "frb_gather_rows_bf16": "pppii",
-    "frb_attention_prefill_tc": "pippipippipppppiiifippipf",
+    "frb_attention_prefill_tc": "pippipippipppppiiifippipf" "iiii",
+    "frb_dyt_rows": "ppppp" "ppp" "pp" "iii" "p" "pppp" "pll",
+    "frb_map_difference": "pppi" "iiiiff",
+    "frb_poly_norm": "pppiiif",
+    "frb_min_gru": "piiii" "pp" "ppp" "pll" "pi" "iii",
+    "frb_retention": "piiiii" "pppp" "pll" "pip" "iiiii" "ff",
     "frb_embed_pair_rows": "pppipiiifillppppppi",
     "frb_token_side_gate": "pppipiiiiii",
     "frb_add_rms_normed": "pppiif",
@@ -87,7 +92,8 @@ _ENTRY_GROUPS = {
     "common": ("frb_embed_rows", "frb_rmsnorm", "frb_qkv_prepare", "frb_add_rows", "frb_attention_generic", "frb_layernorm",
                "frb_unary_unit", "frb_softcap", "frb_gated_unit", "frb_sample_rows", "frb_argmax_rows", "frb_sample_floor",
                "frb_dyt_norm", "frb_rms_blend", "frb_concat_rows", "frb_add_row_vector", "frb_head_gate", "frb_embed_pair_rows",
-               "frb_token_side_gate", "frb_add_rms_normed", "frb_add_typed_copy", "frb_weighted_pair", "frb_sandwich_norm"),
+               "frb_token_side_gate", "frb_add_rms_normed", "frb_add_typed_copy", "frb_weighted_pair", "frb_sandwich_norm",
+               "frb_dyt_rows", "frb_map_difference", "frb_poly_norm"),
     "latent": ("frb_latent_prepare", "frb_latent_queries", "frb_latent_attention", "frb_latent_gate",
                "frb_latent_attention_mma", "frb_latent_attention_tc"),
     "attention": ("frb_attention_decode_mma", "frb_attention_prefill_mma", "frb_attention_decode_tma", "frb_attention_prefill_tc"),
@@ -96,8 +102,10 @@ _ENTRY_GROUPS = {
                 "frb_router_small", "frb_router_logits", "frb_scaled_rows"),
     "products": ("frb_expert_gemm_tc", "frb_gather_rows_bf16"),
     "recurrent": ("frb_gla_scan",),
-    "scans": ("frb_causal_conv", "frb_softplus_bias", "frb_selective_scan", "frb_gated_recurrence", "frb_state_space_scan", "frb_group_rms_norm"),
+    "scans": ("frb_causal_conv", "frb_softplus_bias", "frb_selective_scan", "frb_gated_recurrence", "frb_state_space_scan", "frb_group_rms_norm",
+              "frb_min_gru"),
     "delta": ("frb_gated_delta_rule",),
+    "retention": ("frb_retention",),
     "extras": ("frb_wait_probe",),
 }
 _GROUP_OF = {entry: group for group, entries in _ENTRY_GROUPS.items() for entry in entries}
@@ -394,6 +402,110 @@ def dyt_norm(x: torch.Tensor, first: tuple[torch.Tensor, torch.Tensor, torch.Ten
           _code(out1.dtype), num_rows, x.shape[-1], int(write_back))
 
 
+def _shift_args(shift) -> tuple:
+    """A token shift's (share, ctx, state, offset) as the kernel takes them; nulls without one."""
+    if shift is None:
+        return (None,) * 5 + (None, 0, 0)
+    share, ctx, state, offset = shift
+    _want(share, torch.float32, "a token shift's shares")
+    return (_ptr(share), _ptr(ctx.tok_seq), _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.cu_q_len), *_state_place(state, offset))
+
+
+def dyt_rows(x: torch.Tensor, norm: tuple[torch.Tensor, torch.Tensor, torch.Tensor], out: torch.Tensor, *, deltas: tuple = (),
+             vector: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, stream: Optional[torch.Tensor] = None,
+             shift=None) -> None:
+    """Dynamic tanh of v = x + (d0 + d1 + vector): out = tanh(alpha v) * w + b with ``norm`` = (w, b, alpha).  ``deltas``: up
+    to two float32 tensors [T, width]; ``vector`` [width] is added to every row; ``stream`` gets v (x itself, or another
+    buffer); ``rows`` picks the rows to norm.  ``shift`` = (share, ctx, state, offset): out_t becomes h_t + (h_(t-1) - h_t) *
+    share with h the normed rows, the row before a step's first one coming from the sequence's ``state`` ([slots, 2, floats],
+    this part's at ``offset``), which gets the step's last row; ``stream`` must then be a buffer other than x."""
+    for t in (x, *norm, *deltas):
+        _want(t, torch.float32, "the residual stream, its updates and a dynamic-tanh norm's tensors")
+    deltas = tuple(d for d in deltas if d is not None)
+    if len(deltas) > 2 or any(d.shape != x.shape for d in deltas):
+        raise KernelError("dyt_rows adds at most two tensors of the stream's shape")
+    if vector is not None:
+        _want(vector, torch.float32, "the vector on every row")
+    if rows is not None:
+        _want(rows, torch.int32, "row indices")
+    if stream is not None and (stream.dtype != torch.float32 or stream.shape != x.shape):
+        raise KernelError("dyt_rows: the stream's buffer has another shape or type than the stream")
+    num_rows = rows.numel() if rows is not None else x.shape[0]
+    _call("frb_dyt_rows", _ptr(x), _ptr(deltas[0]) if deltas else None, _ptr(deltas[1]) if len(deltas) > 1 else None, _ptr(vector),
+          _ptr(rows), _ptr(norm[0]), _ptr(norm[1]), _ptr(norm[2]), _ptr(stream), _ptr(out), _code(out.dtype), num_rows, x.shape[-1],
+          *_shift_args(shift))
+
+
+def token_shift(h: torch.Tensor, out: torch.Tensor, *, shift) -> None:
+    """The token shift alone (see :func:`dyt_rows`) on normed float32 rows."""
+    _want(h, torch.float32, "normed rows")
+    _call("frb_dyt_rows", _ptr(h), None, None, None, None, None, None, None, None, _ptr(out), _code(out.dtype), h.shape[0], h.shape[-1],
+          *_shift_args(shift))
+
+
+def map_difference(maps: torch.Tensor, out: torch.Tensor, *, heads: int, kv_heads: int, v_dim: int, lam: torch.Tensor, eps: float,
+                   factor: float) -> None:
+    """``maps`` float32 [T, kv_heads, 2, heads / kv_heads, v_dim]: o = map 1 - lam * map 2 of every head, out [T, heads, v_dim] =
+    o / sqrt(mean(o^2) + eps) * factor."""
+    _want(maps, torch.float32, "the maps' outputs")
+    _want(lam, torch.float32, "lambda")
+    if maps.numel() != 2 * out.numel():
+        raise KernelError("map_difference: the maps' outputs are not twice the output")
+    _call("frb_map_difference", _ptr(maps), _ptr(lam), _ptr(out), _code(out.dtype), out.shape[0], heads, kv_heads, v_dim, float(eps),
+          float(factor))
+
+
+def poly_norm(rows_in: torch.Tensor, coefficients: torch.Tensor, eps: float, out: torch.Tensor) -> None:
+    """out = a N(z) + b N(z^2) + c N(z^3) + e with ``coefficients`` = (a, b, c, e), N(v) = v / sqrt(mean(v^2) + eps) per row."""
+    _want(rows_in, torch.float32, "the activation's input")
+    _want(coefficients, torch.float32, "the activation's coefficients")
+    if coefficients.numel() != 4 or out.shape != rows_in.shape:
+        raise KernelError("poly_norm takes four coefficients and an output of the input's shape")
+    _call("frb_poly_norm", _ptr(rows_in), _ptr(coefficients), _ptr(out), _code(out.dtype), rows_in.shape[0], rows_in.shape[1], float(eps))
+
+
+def min_gru(proj: torch.Tensor, z_offset: int, x_offset: int, g_offset: int, z_bias: torch.Tensor, x_bias: torch.Tensor, ctx,
+            state: torch.Tensor, state_offset: int, out: torch.Tensor) -> None:
+    """z = sigmoid(z + z_bias), u = x + x_bias, cand = u + 1/2 where u >= 0 else sigmoid(u); S <- (1 - z) S + z cand;
+    out = S * silu(g), with z, x and g in float32 columns of ``proj``."""
+    for t in (proj, z_bias, x_bias):
+        _want(t, torch.float32, "min_gru's inputs")
+    _call("frb_min_gru", _ptr(proj), proj.shape[1], int(z_offset), int(x_offset), int(g_offset), _ptr(z_bias), _ptr(x_bias),
+          _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.cu_q_len), *_state_place(state, state_offset), _ptr(out), _code(out.dtype),
+          proj.shape[0], ctx.num_seqs, out.shape[1])
+
+
+RETENTION_CHUNK = 64           # RET_CHUNK of retention.cu: how far its decay tables reach
+
+
+def retention_takes(dim: int, vdim: int) -> bool:
+    """Whether :func:`retention` takes heads of ``dim`` keys and ``vdim`` values (the value columns go over as many blocks as
+    they need)."""
+    return 1 <= dim <= 1024 and vdim >= 1
+
+
+def retention_decays(values, device) -> torch.Tensor:
+    """float32 [heads, 2, RETENTION_CHUNK + 1]: decay^n and decay^n - 1 for n = 0, 1, ..., made in float64, rounded once."""
+    d = torch.tensor([float(v) for v in values], dtype=torch.float64)[:, None]
+    n = torch.arange(RETENTION_CHUNK + 1, dtype=torch.float64)[None, :]
+    powers = torch.pow(d, n)
+    return torch.stack([powers, powers - 1.0], dim=1).to(torch.float32).to(device).contiguous()
+
+
+def retention(proj: torch.Tensor, offsets: tuple[int, int, int, int], decays: torch.Tensor, ctx, state: torch.Tensor, state_offset: int,
+              out: torch.Tensor, raw: torch.Tensor, *, heads: int, dim: int, vdim: int, k_scale: float, eps: float) -> None:
+    """Per head S <- decay S + (k_scale k) v^T, o = S^T q, out = o / sqrt(mean(o^2) + eps) * silu(g): q, k, v, g in float32
+    columns of ``proj`` at the four ``offsets``; ``decays`` as :func:`retention_decays` makes them; ``raw``: float32 scratch of
+    the outputs' size."""
+    for t in (proj, decays, raw):
+        _want(t, torch.float32, "retention's inputs")
+    if raw.numel() < out.numel() or decays.shape[0] != heads or decays.shape[-1] != RETENTION_CHUNK + 1:
+        raise KernelError("retention: the scratch is smaller than the outputs, or the decays are not the heads'")
+    _call("frb_retention", _ptr(proj), proj.shape[1], *(int(o) for o in offsets), _ptr(decays), _ptr(ctx.seq_slot), _ptr(ctx.seq_start),
+          _ptr(ctx.cu_q_len), *_state_place(state, state_offset), _ptr(out), _code(out.dtype), _ptr(raw), proj.shape[0], ctx.num_seqs,
+          int(heads), int(dim), int(vdim), float(k_scale), float(eps))
+
+
 def rms_blend(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch.Tensor, out: torch.Tensor, eps: float,
               share: float) -> None:
     """out = share * (a / rms(a) * wa + b / rms(b) * wb), row by row, all float32."""
@@ -570,13 +682,15 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
                 k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], *, num_heads: int,
                 num_kv_heads: int, head_dim: int, rotary_dim: int, interleaved: bool, write_cache: bool,
                 per_head: bool = False, tables_final: bool = False, bias: Optional[torch.Tensor] = None,
-                v_dim: Optional[int] = None, q_temp: Optional[tuple[float, int]] = None) -> None:
+                v_dim: Optional[int] = None, q_temp: Optional[tuple[float, int]] = None,
+                num_v_heads: Optional[int] = None) -> None:
     """Q/K RMSNorm (when weights are given: over the whole row with weights [heads * head_dim], or with
     ``per_head`` over each head with weights [head_dim]), rotary from the tables, Q out, K/V into their pages.
     ``tables_final``: positions, slots and the page table were complete before the kernel before this one in
     the stream began (a step's tables, with the projection between them and this call); the kernel then reads
     them, and the angles, while that kernel still runs.  ``bias`` (float32, as wide as a row of ``qkv``) is added
-    first; ``v_dim`` is the size of a value head if it is not ``head_dim``; ``q_temp`` = (coef, every) multiplies the
+    first; ``v_dim`` is the size of a value head if it is not ``head_dim``, ``num_v_heads`` their number if it is not
+    ``num_kv_heads``; ``q_temp`` = (coef, every) multiplies the
     query at position p by 1 + coef * ln(floor((p + 1) / every) + 1).  A row without keys and values (a layer that
     reads another layer's cache line) is ``num_kv_heads = 0`` with ``write_cache`` false."""
     if (q_weight is None) != (k_weight is None) and num_kv_heads > 0:
@@ -599,7 +713,8 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
           _ptr(cos_table), _ptr(sin_table), table_positions, _ptr(tok_pos), _ptr(tok_slot), _ptr(page_table), max_pages,
           _ptr(q_out), _ptr(k_pages), _ptr(v_pages), _code(out_dtype), qkv.shape[0], num_heads, num_kv_heads, head_dim,
           rotary_dim, int(interleaved), int(write_cache), int(per_head), int(tables_final), _ptr(bias),
-          int(v_dim or head_dim), float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 1)
+          int(v_dim or head_dim), float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 1,
+          -1 if num_v_heads is None else int(num_v_heads))
 
 
 def attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, page_table: torch.Tensor,
@@ -607,13 +722,14 @@ def attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
                       num_kv_heads: int, head_dim: int, scale: float, window: Optional[int], v_dim: Optional[int] = None,
                       slopes: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
                       sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                      softcap: Optional[float] = None) -> None:
-    """``softcap``: the scaled score s of every key becomes softcap * tanh(s / softcap); ``v_dim``: size of a value head if not ``head_dim``; ``slopes`` (float32 [num_heads]): the score of key j for
+                      softcap: Optional[float] = None, keep_first: int = 0, maps: int = 1) -> None:
+    """``keep_first``: beside the window the sequence's first tokens are visible; ``maps``: that many key heads in a row share a
+    value head; ``softcap``: the scaled score s of every key becomes softcap * tanh(s / softcap); ``v_dim``: size of a value head if not ``head_dim``; ``slopes`` (float32 [num_heads]): the score of key j for
     the query at position i is lowered by slopes[h] * (i - j); ``chunk``: a query sees only the keys of its own chunk
     of that many positions; ``sinks`` (float32 [num_heads]): exp(sinks[h]) joins the softmax's denominator;
     ``gate`` (float32 [T, >= num_heads], rows may be wider): head h's output times sigmoid(gate[t, h])."""
-    if k_pages.dtype != q.dtype or out.dtype != q.dtype:
-        raise KernelError("queries, cache and output must have one dtype")
+    if k_pages.dtype != q.dtype or out.dtype not in (q.dtype, torch.float32):
+        raise KernelError("queries and cache must have one dtype, the output that or float32")
     if slopes is not None:
         _want(slopes, torch.float32, "distance slopes")
     if sinks is not None:
@@ -627,7 +743,8 @@ def attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
     _call("frb_attention_generic", _ptr(q), _ptr(k_pages), _ptr(v_pages), _code(q.dtype), _ptr(page_table),
           page_table.shape[1], _ptr(tok_pos), _ptr(tok_slot), _ptr(out), q.shape[0], num_heads, num_kv_heads, head_dim,
           float(scale), int(window or 0), int(v_dim or head_dim), _ptr(slopes), int(chunk or 0), _ptr(sinks), _ptr(gate),
-          gate.shape[1] if gate is not None else 0, float(softcap or 0.0))
+          gate.shape[1] if gate is not None else 0, float(softcap or 0.0), int(keep_first or 0), num_kv_heads // maps,
+          int(out.dtype == torch.float32))
 
 
 ROUTE_SOFTMAX, ROUTE_FLOOR = 2, 4      # bits of the routing kernels' ``renormalize`` (bit 0: divide by the picked scores' sum)
@@ -825,6 +942,7 @@ def gated_delta_rule(conv: torch.Tensor, q_off: int, k_off: int, v_off: int, pro
 
 
 MMA_HEAD_DIMS = (32, 64, 96, 128)
+MMA_HEAD_SIZES = frozenset({(32, 32), (64, 64), (96, 96), (128, 128), (32, 64), (64, 128)})       # (key head, value head)
 ATTENTION_CHUNK = 256
 
 
@@ -833,8 +951,13 @@ def attention_decode_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
                          out: torch.Tensor, *, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                          window: Optional[int], max_chunks: int, slopes: Optional[torch.Tensor] = None,
                          chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
-                         softcap: Optional[float] = None) -> None:
+                         softcap: Optional[float] = None, v_dim: Optional[int] = None, keep_first: int = 0, maps: int = 1,
+                         difference: Optional[dict] = None) -> None:
     """One token per sequence, bfloat16: keys split into chunks of 256 over blocks, merged in chunk order.
+    ``v_dim`` (here and in the three kernels below): size of a value head if not ``head_dim``; ``keep_first``: beside the window
+    the sequence's first tokens are visible; ``maps``: that many key heads in a row share a value head.  ``difference`` =
+    {lam, eps, factor} (here and in :func:`attention_decode_tma`, with ``maps`` 2): the merge takes the two maps' difference as
+    :func:`map_difference` does.
     ``softcap`` (here and in the three kernels below): the scaled score s becomes softcap * tanh(s / softcap).
     ``slopes`` (float32 [num_heads], here and in the three kernels below): the score of key j for the query at
     position i is lowered by slopes[h] * (i - j); ``chunk``: a query sees only the keys of its own chunk of that many
@@ -844,10 +967,27 @@ def attention_decode_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
     for t in (q, k_pages, v_pages, out):
         _want(t, torch.bfloat16, "tensor-core attention operands")
     _want(part_o, torch.float32, "partial outputs")
+    lam, eps, factor = _difference_args(difference, maps)
     _call("frb_attention_decode_mma", _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(page_table), page_table.shape[1],
           _ptr(seq_pos), _ptr(seq_slot), _ptr(part_o), _ptr(part_ml), _ptr(out), q.shape[0], num_heads, num_kv_heads,
           head_dim, float(scale), int(window or 0), max_chunks, _ptr(tc_status(q.device)), _ptr(slopes), int(chunk or 0),
-          _ptr(sinks), float(softcap or 0.0))
+          _ptr(sinks), float(softcap or 0.0), int(v_dim or head_dim), int(keep_first or 0), num_kv_heads // maps, lam, eps, factor)
+
+
+def _difference_args(difference: Optional[dict], maps: int) -> tuple:
+    if difference is None:
+        return None, 0.0, 0.0
+    if maps != 2:
+        raise KernelError(f"the difference of {maps} maps")
+    _want(difference["lam"], torch.float32, "lambda")
+    return _ptr(difference["lam"]), float(difference["eps"]), float(difference["factor"])
+
+
+def _maps_output(out: torch.Tensor) -> int:
+    """Whether a prompt kernel writes float32 (bfloat16 otherwise)."""
+    if out.dtype not in (torch.bfloat16, torch.float32):
+        raise KernelError(f"an attention output of {out.dtype}")
+    return int(out.dtype == torch.float32)
 
 
 def _want_slopes(slopes: Optional[torch.Tensor], num_heads: int) -> None:
@@ -889,8 +1029,9 @@ def attention_decode_tma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
                          out: torch.Tensor, *, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                          window: Optional[int], max_chunks: int, chunks_per_block: Optional[int] = None,
                          slopes: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                         sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
-    """As :func:`attention_decode_mma` for head sizes 64 and 128, with the pages copied into shared memory by
+                         sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None, v_dim: Optional[int] = None,
+                         keep_first: int = 0, maps: int = 1, difference: Optional[dict] = None) -> None:
+    """As :func:`attention_decode_mma` for key heads of 64 and 128, with the pages copied into shared memory by
     TMA through a ring of stages, which keeps far more bytes in flight; a block takes ``chunks_per_block``
     chunks (default: :func:`decode_chunks_per_block`)."""
     for t in (q, k_pages, v_pages, out):
@@ -900,10 +1041,12 @@ def attention_decode_tma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
     _want_slopes(sinks, num_heads)
     if chunks_per_block is None:
         chunks_per_block = decode_chunks_per_block(q.shape[0], num_kv_heads, max_chunks, sm_count(q.device))
+    lam, eps, factor = _difference_args(difference, maps)
     _call("frb_attention_decode_tma", _ptr(q), _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(page_table),
           page_table.shape[1], _ptr(seq_pos), _ptr(seq_slot), _ptr(part_o), _ptr(part_ml), _ptr(out), q.shape[0], num_heads,
           num_kv_heads, head_dim, float(scale), int(window or 0), max_chunks, int(chunks_per_block),
-          _ptr(tc_status(q.device)), _ptr(slopes), int(chunk or 0), _ptr(sinks), float(softcap or 0.0))
+          _ptr(tc_status(q.device)), _ptr(slopes), int(chunk or 0), _ptr(sinks), float(softcap or 0.0), int(v_dim or head_dim),
+          int(keep_first or 0), num_kv_heads // maps, lam, eps, factor)
 
 
 def attention_prefill_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, page_table: torch.Tensor,
@@ -911,16 +1054,18 @@ def attention_prefill_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch
                           seq_q_len: torch.Tensor, cu_q_len: torch.Tensor, out: torch.Tensor, *, num_heads: int,
                           num_kv_heads: int, head_dim: int, scale: float, window: Optional[int],
                           slopes: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                          sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
-    """Many tokens per sequence, bfloat16: tiles of 16 queries, causal, blockwise over the cache pages."""
-    for t in (q, k_pages, v_pages, out):
+                          sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None, v_dim: Optional[int] = None,
+                          keep_first: int = 0, maps: int = 1) -> None:
+    """Many tokens per sequence, bfloat16 (the output in that or float32): tiles of 16 queries, causal, blockwise over the cache pages."""
+    for t in (q, k_pages, v_pages):
         _want(t, torch.bfloat16, "tensor-core attention operands")
     _want_slopes(slopes, num_heads)
     _want_slopes(sinks, num_heads)
     _call("frb_attention_prefill_mma", _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(page_table), page_table.shape[1],
           _ptr(tile_seq), _ptr(tile_q0), tile_seq.numel(), _ptr(seq_slot), _ptr(seq_start), _ptr(seq_q_len),
           _ptr(cu_q_len), _ptr(out), num_heads, num_kv_heads, head_dim, float(scale), int(window or 0), _ptr(slopes),
-          int(chunk or 0), _ptr(sinks), float(softcap or 0.0))
+          int(chunk or 0), _ptr(sinks), float(softcap or 0.0), int(v_dim or head_dim), int(keep_first or 0), num_kv_heads // maps,
+          _maps_output(out))
 
 
 def expert_gemm_mma(w: torch.Tensor, x: torch.Tensor, x_rows: Optional[torch.Tensor], tile_expert: torch.Tensor,
@@ -1118,17 +1263,19 @@ def attention_prefill_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
                          seq_q_len: torch.Tensor, cu_q_len: torch.Tensor, out: torch.Tensor, *, num_heads: int,
                          num_kv_heads: int, head_dim: int, scale: float, window: Optional[int],
                          slopes: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                         sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
-    """Many tokens per sequence on tcgen05 tensor cores: tiles of 128 queries of one head (bfloat16, head sizes
-    64 and 128).  Capped scores and distance slopes together are refused."""
-    for t in (q, k_pages, v_pages, out):
+                         sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None, v_dim: Optional[int] = None,
+                         keep_first: int = 0, maps: int = 1) -> None:
+    """Many tokens per sequence on tcgen05 tensor cores: tiles of 128 queries of one head (bfloat16, the output in that or
+    float32; key heads of 64 and 128).  Capped scores and distance slopes together are refused."""
+    for t in (q, k_pages, v_pages):
         _want(t, torch.bfloat16, "tensor-core attention operands")
     _want_slopes(slopes, num_heads)
     _want_slopes(sinks, num_heads)
     _call("frb_attention_prefill_tc", _ptr(q), q.shape[0], _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(page_table),
           page_table.shape[1], _ptr(tile_seq), _ptr(tile_q0), tile_seq.numel(), _ptr(seq_slot), _ptr(seq_start),
           _ptr(seq_q_len), _ptr(cu_q_len), _ptr(out), num_heads, num_kv_heads, head_dim, float(scale), int(window or 0),
-          _ptr(tc_status(q.device)), _ptr(slopes), int(chunk or 0), _ptr(sinks), float(softcap or 0.0))
+          _ptr(tc_status(q.device)), _ptr(slopes), int(chunk or 0), _ptr(sinks), float(softcap or 0.0), int(v_dim or head_dim),
+          int(keep_first or 0), num_kv_heads // maps, _maps_output(out))
 
 
 def wait_probe(device, limit_cycles: int = 100_000) -> int:

@@ -6,6 +6,7 @@
 //   selective_scan   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n;  y_c = sum_n S[c, n] C_n + D_c x_c;  y silu(z)
 //   gated_recurrence a = exp(-g r softplus(lam)),  S <- a S + sqrt(1 - a^2) i u,  out = S * act(y)    (per channel)
 //   state_space_scan per head: S <- exp(-exp(A_log) dt) S + dt B x^T (S is [N, vdim]);  y = S^T C + D x;  y silu(z)
+//   min_gru          z = sigmoid(z + bz), u = x + bx, cand = u >= 0 ? u + 1/2 : sigmoid(u);  S <- (1 - z) S + z cand;  out = S silu(g)
 //   group_rms_norm   rows divided, in equal parts, by each part's root mean square, times a weight
 //
 // Everything here is float32: the rows come as the float32 results of the projections, the state lives in float32.
@@ -613,6 +614,125 @@ FRB_API int frb_state_space_scan(const float* proj, int proj_stride, int z_offse
     else FRB_SSD(64, 1);
 #undef FRB_SSD
     FRB_RETURN_LAUNCH("state_space_scan");
+}
+
+// ---------------------------------------------------------------------------------------------------- min_gru
+
+#define GRU_WARPS 16         // runs of tokens that a block takes side by side
+#define GRU_TOKENS 8         // tokens of a run
+
+struct MinGruParams {
+    const float* proj;       // [T, proj_stride]: z of channel c at z_offset + c, x at x_offset + c, the gate at g_offset + c, before biases
+    const float* z_bias;     // [C]
+    const float* x_bias;     // [C]
+    SeqTables seq;
+    StatePlace state;        // [C]
+    void* out;               // [T, C]
+    int proj_stride, z_offset, x_offset, g_offset, channels;
+};
+
+// One token's step S <- (1 - z) S + z cand as S <- coef S + (fresh ? 0 : S) + input.  With z below a half coef = -z (the share
+// that leaves: 1 - z rounded to float32 would lose its distance from one by the same amount at every token), else
+// coef = 1 - z itself, made without a subtraction.
+struct GruStep { float coef, input; bool fresh; };
+
+__device__ __forceinline__ GruStep gru_step(float z_logit, float u) {
+    const float e = expf(-fabsf(z_logit)), big = 1.0f / (1.0f + e), small = e * big;      // sigmoid(|l|), sigmoid(-|l|)
+    GruStep s;
+    s.fresh = z_logit > 0.f;
+    const float z = s.fresh ? big : small;
+    s.coef = s.fresh ? small : -small;
+    s.input = z * (u >= 0.f ? u + 0.5f : sigmoid_f(u));
+    return s;
+}
+__device__ __forceinline__ float gru_apply(const GruStep& s, float S) { return fmaf(s.coef, S, s.fresh ? 0.f : S) + s.input; }
+
+// One token a sequence: a thread per (sequence, channel).
+template <typename OutT>
+__global__ void __launch_bounds__(128) min_gru_token_kernel(MinGruParams p) {
+    after_previous_kernel();
+    const int c = blockIdx.x * 128 + threadIdx.x, b = blockIdx.y;
+    if (c >= p.channels) return;
+    const int row = p.seq.cu_q_len[b], start = p.seq.seq_start[b], slot = p.seq.seq_slot[b];
+    const float* in = p.proj + (size_t)row * p.proj_stride + c;
+    const float l = in[p.z_offset] + p.z_bias[c], u = in[p.x_offset] + p.x_bias[c], g = in[p.g_offset];
+    const float S = gru_apply(gru_step(l, u), state_at(p.state, slot, start & 1)[c]);
+    state_at(p.state, slot, (start + 1) & 1)[c] = S;
+    ((OutT*)p.out)[(size_t)row * p.channels + c] = from_f32<OutT>(S * silu_for<OutT>(g));
+}
+
+// Prompts: a block takes 32 channels (one a lane) of one sequence, GRU_WARPS x GRU_TOKENS tokens at a time.  Each warp makes
+// its run's steps, side by side with the others, and what the run as a whole does to a state: S <- S + less * S + sum, `less`
+// being the product of its decays less one.  Behind one barrier every warp goes through the runs before its own to find its
+// first state, then takes its tokens one by one from there; the last warp's state is the next round's first.
+template <typename OutT>
+__global__ void __launch_bounds__(32 * GRU_WARPS) min_gru_kernel(MinGruParams p) {
+    __shared__ float s_less[2][GRU_WARPS][32], s_sum[2][GRU_WARPS][32], s_first[2][32];
+    after_previous_kernel();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, b = blockIdx.y;
+    const int c = blockIdx.x * 32 + lane;
+    const bool live = c < p.channels;
+    const int row0 = p.seq.cu_q_len[b], n_tok = p.seq.cu_q_len[b + 1] - row0;
+    const int start = p.seq.seq_start[b], slot = p.seq.seq_slot[b];
+    const float z_bias = live ? p.z_bias[c] : 0.f, x_bias = live ? p.x_bias[c] : 0.f;
+    float S = live && warp == 0 ? state_at(p.state, slot, start & 1)[c] : 0.f;
+    if (warp == 0) s_first[0][lane] = S;
+    OutT* out = (OutT*)p.out;
+    int round = 0;
+    for (int t0 = 0; t0 < n_tok; t0 += GRU_WARPS * GRU_TOKENS, ++round) {
+        const int mine = t0 + warp * GRU_TOKENS, now = round & 1;
+        float zl[GRU_TOKENS], ul[GRU_TOKENS], gl[GRU_TOKENS];
+#pragma unroll
+        for (int i = 0; i < GRU_TOKENS; ++i) {
+            const bool has = live && mine + i < n_tok;
+            const float* in = p.proj + (size_t)(row0 + mine + i) * p.proj_stride + c;
+            zl[i] = has ? in[p.z_offset] + z_bias : 0.f;
+            ul[i] = has ? in[p.x_offset] + x_bias : 0.f;
+            gl[i] = has ? in[p.g_offset] : 0.f;
+        }
+        GruStep step[GRU_TOKENS];
+        float less = 0.f, sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < GRU_TOKENS; ++i) {
+            if (mine + i < n_tok) step[i] = gru_step(zl[i], ul[i]);
+            else step[i] = GruStep{0.f, 0.f, false};                     // a token that is not there leaves the state as it is
+            const float leaves = step[i].fresh ? step[i].coef - 1.0f : step[i].coef;
+            less = fmaf(leaves, less, leaves + less);                    // (1 + leaves)(1 + less) - 1
+            sum = gru_apply(step[i], sum);
+        }
+        s_less[now][warp][lane] = less;
+        s_sum[now][warp][lane] = sum;
+        __syncthreads();             // the other copies of these arrays are free: all warps have come here, and read them before
+        S = s_first[now][lane];
+        for (int w = 0; w < warp; ++w) S = fmaf(s_less[now][w][lane], S, S) + s_sum[now][w][lane];
+#pragma unroll
+        for (int i = 0; i < GRU_TOKENS; ++i) {
+            S = gru_apply(step[i], S);
+            if (live && mine + i < n_tok)
+                out[(size_t)(row0 + mine + i) * p.channels + c] = from_f32<OutT>(S * silu_for<OutT>(gl[i]));
+        }
+        if (warp == GRU_WARPS - 1) s_first[now ^ 1][lane] = S;
+    }
+    if (live && warp == GRU_WARPS - 1) state_at(p.state, slot, (start + n_tok) & 1)[c] = S;
+}
+
+FRB_API int frb_min_gru(const float* proj, int proj_stride, int z_offset, int x_offset, int g_offset, const float* z_bias,
+                        const float* x_bias, const int* seq_slot, const int* seq_start, const int* cu_q_len, float* state,
+                        long long copy_floats, long long state_offset, void* out, int out_dtype, int num_rows, int num_seqs,
+                        int channels, cudaStream_t stream) {
+    if (num_seqs == 0) return 0;
+    FRB_CHECK_ARG(num_seqs <= 65535, "min_gru: %d sequences exceed the grid", num_seqs);
+    MinGruParams p;
+    p.proj = proj; p.z_bias = z_bias; p.x_bias = x_bias; p.seq = SeqTables{seq_slot, seq_start, cu_q_len};
+    p.state = StatePlace{state, copy_floats, state_offset};
+    p.out = out; p.proj_stride = proj_stride; p.z_offset = z_offset; p.x_offset = x_offset; p.g_offset = g_offset; p.channels = channels;
+    FRB_DISPATCH_DTYPE(out_dtype, OutT, {
+        if (num_rows == num_seqs)
+            launch_dependent(min_gru_token_kernel<OutT>, dim3((channels + 127) / 128, num_seqs), dim3(128), 0, stream, p);
+        else
+            launch_dependent(min_gru_kernel<OutT>, dim3((channels + 31) / 32, num_seqs), dim3(32 * GRU_WARPS), 0, stream, p);
+    });
+    FRB_RETURN_LAUNCH("min_gru");
 }
 
 // ---------------------------------------------------------------------------------------------------- group_rms_norm

@@ -50,6 +50,9 @@ class DecoderModel:
                 build_part("norm", layer.feed_forward_norm, self.dtype) if layer.feed_forward_norm is not None else None,
                 build_part("norm", layer.mixer_out_norm, self.dtype) if layer.mixer_out_norm is not None else None,
                 build_part("norm", layer.feed_forward_out_norm, self.dtype) if layer.feed_forward_out_norm is not None else None))
+        for block, layer in zip(self.blocks, plan.layers):
+            if layer.mixer_input is not None:
+                block.set_mixer_input(build_part("mixer_input", layer.mixer_input, self.dtype))
         self.additions = [build_part("addition", layer.addition, self.dtype) if layer.addition is not None else None
                           for layer in plan.layers]
         self.connectors = [build_part("connector", spec, self.dtype) for spec in plan.connectors]
@@ -132,7 +135,7 @@ class DecoderModel:
         lines = max((run.cache_line for run in self.plan.run_order), default=-1) + 1
         needs: list[Optional[CacheNeed]] = [None] * lines
         for run in self.plan.run_order:
-            need = self.blocks[run.layer].mixer.cache_need()
+            need = self.blocks[run.layer].cache_need()
             if run.writes_cache:
                 needs[run.cache_line] = need
             elif needs[run.cache_line] != need:
@@ -172,7 +175,7 @@ class DecoderModel:
         pending = None
         for run in self.plan.run_order:
             if run.connector is not None:
-                x, pending = self.connectors[run.connector[0]].forward(ctx, x, pending, first, run.connector[1]), None
+                x, pending = self.connectors[run.connector[0]].forward_deferred(ctx, x, pending, first, run.connector[1])
             x, pending = self.blocks[run.layer].forward(ctx, x, pending, cache.line(run.cache_line), run.writes_cache)
             if self.additions[run.layer] is not None:
                 x, pending = self.additions[run.layer].forward(ctx, x, pending)

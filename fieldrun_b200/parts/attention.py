@@ -22,7 +22,18 @@ before the current chunk), ``sink`` (a learned number per query head whose expon
 denominator: no key, no value, not scaled, counted once), ``head_gate`` (head h's output is multiplied by
 sigmoid(W_g x)_h, one row of W_g per head, before the output projection), ``sink_value`` (the sink as a constant for
 every head instead of a learned tensor: 0.0 adds one to the softmax's denominator), ``softcap`` (the scaled score s
-of every key becomes softcap * tanh(s / softcap) before the softmax).
+of every key becomes softcap * tanh(s / softcap) before the softmax), ``keep_first`` (beside a window, the sequence's first
+tokens stay visible to every query, at their true positions; the cache keeps their pages), ``output_bias`` (the output
+projection has a bias, left to the norm that takes the update), ``differential`` ``{"diff", "eps"}``: every head has two maps,
+each an attention of its own with queries and keys of ``head_dim`` over the same values, and gives
+
+    o = a1 - lambda a2,   out = o / sqrt(mean(o^2) + eps) * (1 - diff)   (over the head's value entries),
+    lambda = exp(sum(lq1 * lk1)) - exp(sum(lq2 * lk2)) + diff            (four learned vectors of head_dim, one lambda a layer).
+
+A projection's rows are laid out head by head as [map 1, map 2]; the kernels see the two maps as query heads and key heads of
+their own (rows are put into the order key head, map, query head of the group at load), two key heads sharing a value head.
+The difference is taken in float32: of the one-token kernels' partial results where those are joined, of float32 outputs
+otherwise.
 """
 from __future__ import annotations
 
@@ -33,7 +44,7 @@ import torch
 from ..cache import CacheNeed, LineView
 from ..csrc import ops
 from ..weights.loader import MATRIX, VECTOR, TensorNeed, TensorSource
-from .base import Mixer, build_position, register_part
+from .base import BiasedRows, Mixer, build_position, register_part
 from .linear import linear
 
 
@@ -84,6 +95,19 @@ class GQAAttention(Mixer):
         self.has_head_gate = bool(a.get("head_gate", False))
         self.sinks: Optional[torch.Tensor] = None
         self.w_gate: Optional[torch.Tensor] = None
+        self.keep_first = int(a.get("keep_first") or 0) if self.window is not None else 0
+        if self.keep_first and self.chunk is not None:
+            raise ValueError("first tokens that stay visible go with a window, not with chunks")
+        self.has_output_bias = bool(a.get("output_bias", False))
+        self.b_o: Optional[torch.Tensor] = None
+        differential = a.get("differential")
+        self.maps = 2 if differential else 1
+        self.diff = float(differential["diff"]) if differential else 0.0
+        self.diff_eps = float(differential.get("eps", 1e-6)) if differential else 0.0
+        self.lam: Optional[torch.Tensor] = None
+        if differential and (self.qk_norm != "none" or self.shares_kv or self.has_head_gate or self.has_sink
+                             or self.sink_value is not None or self.slope_values is not None):
+            raise ValueError("differential attention is built without q/k norms, shared keys, head gates, sinks and distance slopes")
         if self.num_heads % self.num_kv_heads:
             raise ValueError(f"{self.num_heads} heads are not a multiple of {self.num_kv_heads} kv heads")
         if not 1 <= self.head_dim <= 256:
@@ -93,10 +117,13 @@ class GQAAttention(Mixer):
         self.position = build_position(a.get("position"))
         if self.position is not None and self.position.rotary_dim > self.head_dim:
             raise ValueError(f"rotary_dim {self.position.rotary_dim} exceeds head_dim {self.head_dim}")
-        if not (dtype == torch.bfloat16 and self.value_dim == self.head_dim and self.head_dim in ops.MMA_HEAD_DIMS):
+        self.tensor_cores = dtype == torch.bfloat16 and (self.head_dim, self.value_dim) in ops.MMA_HEAD_SIZES
+        if not self.tensor_cores:
             self.kernel_groups = ("common", "streams")          # the tensor-core kernels take none of this part's steps
-        self.q_width = self.num_heads * self.head_dim
-        self.kv_width = self.num_kv_heads * self.head_dim
+        # heads as the kernels see them: with two maps per head, two query heads and two key heads
+        self.q_heads, self.k_heads = self.maps * self.num_heads, self.maps * self.num_kv_heads
+        self.q_width = self.q_heads * self.head_dim
+        self.kv_width = self.k_heads * self.head_dim
         self.v_width = self.num_kv_heads * self.value_dim
         self.out_width = self.num_heads * self.value_dim
         self.b_qkv: Optional[torch.Tensor] = None
@@ -119,6 +146,11 @@ class GQAAttention(Mixer):
             needs["q_bias"] = TensorNeed(self.name_of("q_bias"), (self.q_width,), VECTOR, "bias")
             needs["k_bias"] = TensorNeed(self.name_of("k_bias"), (self.kv_width,), VECTOR, "bias")
             needs["v_bias"] = TensorNeed(self.name_of("v_bias"), (self.v_width,), VECTOR, "bias")
+        if self.has_output_bias:
+            needs["o_bias"] = TensorNeed(self.name_of("o_bias"), (self.hidden_size,), VECTOR, "bias")
+        if self.maps == 2:
+            for local in ("lambda_q1", "lambda_k1", "lambda_q2", "lambda_k2"):
+                needs[local] = TensorNeed(self.name_of(local), (self.head_dim,), VECTOR, "around_zero")
         if self.qk_norm == "full_width":
             needs["q_norm"] = TensorNeed(self.name_of("q_norm"), (self.q_width,), VECTOR, "around_one")
             needs["k_norm"] = TensorNeed(self.name_of("k_norm"), (self.kv_width,), VECTOR, "around_one")
@@ -140,11 +172,16 @@ class GQAAttention(Mixer):
     def load(self, source: TensorSource) -> None:
         needs = self._needs()
         projections = ("q_proj",) if self.shares_kv else ("q_proj", "k_proj", "v_proj")
-        self.w_qkv = torch.cat([source.fetch(needs[n]) for n in projections], dim=0).contiguous()
+        self.w_qkv = torch.cat([self._map_order(n, source.fetch(needs[n])) for n in projections], dim=0).contiguous()
         self.w_o = source.fetch(needs["o_proj"])
         if self.has_bias:
             biases = ("q_bias",) if self.shares_kv else ("q_bias", "k_bias", "v_bias")
-            self.b_qkv = torch.cat([source.fetch(needs[n]) for n in biases], dim=0).contiguous()
+            self.b_qkv = torch.cat([self._map_order(n, source.fetch(needs[n])) for n in biases], dim=0).contiguous()
+        if self.has_output_bias:
+            self.b_o = source.fetch(needs["o_bias"])
+        if self.maps == 2:
+            q1, k1, q2, k2 = (source.fetch(needs[n]).double() for n in ("lambda_q1", "lambda_k1", "lambda_q2", "lambda_k2"))
+            self.lam = (torch.exp((q1 * k1).sum()) - torch.exp((q2 * k2).sum()) + self.diff).to(torch.float32).reshape(1)
         if self.has_sink:
             self.sinks = source.fetch(needs["sink"])
         if self.has_head_gate:
@@ -153,9 +190,19 @@ class GQAAttention(Mixer):
             self.q_norm = source.fetch(needs["q_norm"])
             self.k_norm = source.fetch(needs["k_norm"]) if "k_norm" in needs else None
 
+    def _map_order(self, name: str, rows: torch.Tensor) -> torch.Tensor:
+        """The query projection's rows (or bias) in the kernels' order of heads: [key head, map, query head of the group]
+        instead of [key head, query head of the group, map].  Keys and values are in order as they are."""
+        if self.maps == 1 or not name.startswith("q_"):
+            return rows
+        group = self.num_heads // self.num_kv_heads
+        shaped = rows.reshape(self.num_kv_heads, group, self.maps, self.head_dim, *rows.shape[1:])
+        return shaped.transpose(1, 2).reshape(rows.shape)
+
     # -- cache and tables ----------------------------------------------------------------------------
     def cache_need(self) -> CacheNeed:
-        return CacheNeed(kv_heads=self.num_kv_heads, head_dim=self.head_dim,
+        return CacheNeed(kv_heads=self.k_heads, head_dim=self.head_dim, keep_first=self.keep_first,
+                         value_heads=self.num_kv_heads if self.maps == 2 else 0,
                          window=int(self.window) if self.window is not None else None,
                          value_dim=self.value_dim if self.value_dim != self.head_dim else 0, chunk=self.chunk)
 
@@ -176,8 +223,9 @@ class GQAAttention(Mixer):
         q = ctx.buffer("attention.q", (tokens, self.q_width), self.dtype)
         rotary_dim = self.position.rotary_dim if self.position is not None else 0
         ops.qkv_prepare(qkv, self.q_norm, self.k_norm, self.qk_norm_eps, self.cos, self.sin, ctx.tok_pos, ctx.tok_slot,
-                        line.page_table, q, line.keys, line.values, num_heads=self.num_heads,
-                        num_kv_heads=0 if self.shares_kv else self.num_kv_heads, head_dim=self.head_dim,
+                        line.page_table, q, line.keys, line.values, num_heads=self.q_heads,
+                        num_kv_heads=0 if self.shares_kv else self.k_heads, num_v_heads=0 if self.shares_kv else self.num_kv_heads,
+                        head_dim=self.head_dim,
                         rotary_dim=rotary_dim,
                         interleaved=bool(self.position.interleaved) if self.position is not None else False,
                         write_cache=writes_cache, per_head=self.qk_norm == "per_head",
@@ -186,40 +234,46 @@ class GQAAttention(Mixer):
         out = ctx.buffer("attention.out", (tokens, self.out_width), self.dtype)
         gate = linear(act, self.w_gate) if self.has_head_gate else None          # float32 [T, heads], before the sigmoid
         self.attend(ctx, q, line, out, gate)
-        return linear(out, self.w_o)
+        update = linear(out, self.w_o)
+        return BiasedRows(update, self.b_o) if self.b_o is not None else update
 
     def attend(self, ctx, q: torch.Tensor, line: LineView, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> None:
-        """Tensor-core kernels for bfloat16 and head sizes of 32, 64, 96 or 128 (tcgen05 for prompts with head
-        sizes 64 and 128, mma.sync otherwise), keys and values of one size; the general kernel for everything else.
-        All of them take the distance slopes, chunks and sinks; the general kernel applies the head gates itself, after
-        the others a small kernel does."""
-        common = dict(num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, head_dim=self.head_dim,
+        """Tensor-core kernels for bfloat16 and the head sizes of ``ops.MMA_HEAD_SIZES`` (tcgen05 for prompts with key
+        heads of 64 and 128, mma.sync otherwise); the general kernel for everything else.  All of them take the distance
+        slopes, chunks, sinks and first tokens; the general kernel applies the head gates itself, after the others a small
+        kernel does.  With two maps per head the one-token kernels take the maps' difference where they join their partial
+        results, after the others a small kernel does."""
+        common = dict(num_heads=self.q_heads, num_kv_heads=self.k_heads, head_dim=self.head_dim, v_dim=self.value_dim,
                       scale=self.softmax_scale, window=self.window, slopes=self.slopes, chunk=self.chunk, sinks=self.sinks,
-                      softcap=self.softcap)
+                      softcap=self.softcap, keep_first=self.keep_first, maps=self.maps)
+        difference = dict(lam=self.lam, eps=self.diff_eps, factor=1.0 - self.diff)
         both = self.softcap is not None and self.slopes is not None     # the tcgen05 kernel has either, not both
-        if self.value_dim == self.head_dim and self.dtype == torch.bfloat16 and self.head_dim in ops.MMA_HEAD_DIMS and not both:
+        maps_out = out if self.maps == 1 else ctx.buffer("attention.maps", (out.shape[0], self.maps * self.out_width), torch.float32)
+        if self.tensor_cores and not both:
             if ctx.is_decode and self.num_heads // self.num_kv_heads <= 16:
                 chunks = (ctx.max_kv_len + ops.ATTENTION_CHUNK - 1) // ops.ATTENTION_CHUNK
-                part_o = ctx.buffer("attention.part_o", (ctx.num_seqs, self.num_heads, chunks, self.head_dim), torch.float32)
-                part_ml = ctx.buffer("attention.part_ml", (ctx.num_seqs, self.num_heads, chunks, 2), torch.float32)
+                part_o = ctx.buffer("attention.part_o", (ctx.num_seqs, self.q_heads, chunks, self.value_dim), torch.float32)
+                part_ml = ctx.buffer("attention.part_ml", (ctx.num_seqs, self.q_heads, chunks, 2), torch.float32)
                 # head sizes 64 and 128: the pages come into shared memory by TMA; others: loads into registers
                 decode = ops.attention_decode_tma if self.head_dim in ops.TC_ATTENTION_HEAD_DIMS else ops.attention_decode_mma
                 decode(q, line.keys, line.values, line.page_table, ctx.seq_start, ctx.seq_slot, part_o, part_ml, out,
-                       max_chunks=chunks, **common)
+                       max_chunks=chunks, difference=difference if self.maps == 2 else None, **common)
+                maps_out = out
             elif self.head_dim in ops.TC_ATTENTION_HEAD_DIMS and ctx.max_q_len >= TC_ATTENTION_MIN_QUERIES:
                 # prompts: 128 queries of one head per block, both products on tcgen05
                 tile_seq, tile_q0 = ctx.query_tiles(ops.TC_ATTENTION_QUERIES)
                 ops.attention_prefill_tc(q, line.keys, line.values, line.page_table, tile_seq, tile_q0, ctx.seq_slot,
-                                         ctx.seq_start, ctx.seq_q_len, ctx.cu_q_len, out, **common)
+                                         ctx.seq_start, ctx.seq_q_len, ctx.cu_q_len, maps_out, **common)
             else:
                 tile_seq, tile_q0 = ctx.query_tiles(16)
                 ops.attention_prefill_mma(q, line.keys, line.values, line.page_table, tile_seq, tile_q0, ctx.seq_slot,
-                                          ctx.seq_start, ctx.seq_q_len, ctx.cu_q_len, out, **common)
+                                          ctx.seq_start, ctx.seq_q_len, ctx.cu_q_len, maps_out, **common)
             if gate is not None:
                 ops.head_gate(out, gate, self.num_heads, self.value_dim)
-            return
-        ops.attention_generic(q, line.keys, line.values, line.page_table, ctx.tok_pos, ctx.tok_slot, out,
-                              v_dim=self.value_dim, gate=gate, **common)
+        else:
+            ops.attention_generic(q, line.keys, line.values, line.page_table, ctx.tok_pos, ctx.tok_slot, maps_out, gate=gate, **common)
+        if maps_out is not out:
+            ops.map_difference(maps_out, out, heads=self.num_heads, kv_heads=self.num_kv_heads, v_dim=self.value_dim, **difference)
 
 
 register_part("mixer", "gqa_attention", GQAAttention, replace=True)

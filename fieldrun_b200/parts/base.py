@@ -24,6 +24,9 @@ Interfaces
     a norm behind a sublayer whose block also has one in front (``NormedUpdate`` carries the pair to the next norm).
 ``Connector.forward(ctx, x, pending, first, index)`` -> the new stream [T, width] (float32)
     a part between two runs that rewrites the whole stream; ``first`` holds the embedding's rows.
+    ``forward_deferred`` -> (stream, pending): for one that only adds and may leave the sum to the next norm.
+``MixerInput.forward(ctx, norm, x, pending, line, offset)`` -> (x, act)
+    a part between the mixer's norm and the mixer: it runs the norm and gives the rows that the mixer reads.
 ``Addition.forward(ctx, x, pending)`` -> (x, pending)
     a part behind a layer's block that adds to the stream once more (a further input per layer and token).
 """
@@ -105,18 +108,33 @@ class WeightedRows(DeferredUpdate):
         return out
 
 
+class BiasedRows(DeferredUpdate):
+    """A float32 tensor [T, width] and a vector [width] that every row of it still has to get (the bias of a projection
+    that ends a sublayer), so that the norm which takes the update can add it while it reads the rows."""
+
+    def __init__(self, rows: torch.Tensor, vector: torch.Tensor):
+        self.rows, self.vector = rows, vector
+
+    def materialize(self, ctx) -> torch.Tensor:
+        from ..csrc import ops
+        ops.add_row_vector(self.rows, self.vector, self.rows)
+        return self.rows
+
+
 class UpdateSum(DeferredUpdate):
-    """Several updates of one stream that are added together: float32 tensors [T, width] and at most one
-    :class:`WeightedRows`.  A block whose sublayers all read the same x leaves their outputs in this form, so
-    that the norm which reads the stream next adds them while it reads (a norm that does not know the form
-    gets their sum from ``materialize``)."""
+    """Several updates of one stream that are added together: float32 tensors [T, width], at most one
+    :class:`WeightedRows` and at most one :class:`BiasedRows`.  A block whose sublayers all read the same x leaves their
+    outputs in this form, so that the norm which reads the stream next adds them while it reads (a norm that does not
+    know the form gets their sum from ``materialize``)."""
 
     def __init__(self, updates):
-        self.tensors = [u for u in updates if isinstance(u, torch.Tensor)]
+        biased = [u for u in updates if isinstance(u, BiasedRows)]
+        self.tensors = [u.rows if isinstance(u, BiasedRows) else u for u in updates if isinstance(u, (torch.Tensor, BiasedRows))]
+        self.vector = biased[0].vector if biased else None
         self.weighted = [u for u in updates if isinstance(u, WeightedRows)]
-        other = [u for u in updates if u is not None and not isinstance(u, (torch.Tensor, WeightedRows))]
-        if other or len(self.weighted) > 1:
-            raise ValueError("an UpdateSum holds float32 tensors and at most one WeightedRows")
+        other = [u for u in updates if u is not None and not isinstance(u, (torch.Tensor, WeightedRows, BiasedRows))]
+        if other or len(self.weighted) > 1 or len(biased) > 1:
+            raise ValueError("an UpdateSum holds float32 tensors, at most one WeightedRows and at most one BiasedRows")
 
     def materialize(self, ctx) -> torch.Tensor:
         from ..csrc import ops
@@ -126,6 +144,8 @@ class UpdateSum(DeferredUpdate):
                 total = update
             else:
                 ops.add_rows(total, update)
+        if self.vector is not None:
+            ops.add_row_vector(total, self.vector, total)
         return total
 
 
@@ -228,6 +248,21 @@ class Connector(Part):
     def forward(self, ctx, x: torch.Tensor, pending, first: torch.Tensor, index: int) -> torch.Tensor:
         raise NotImplementedError
 
+    def forward_deferred(self, ctx, x: torch.Tensor, pending, first: torch.Tensor, index: int):
+        """Like ``forward``, but returns (stream, pending) and may leave an addition to the next norm."""
+        return self.forward(ctx, x, pending, first, index), None
+
+
+class MixerInput(Part):
+    """A part between a mixer's norm and the mixer.  It may keep a float32 state per sequence, twice (``state_floats``
+    floats behind the mixer's own state, see ``CacheNeed.with_state_behind``; ``offset`` says where they begin)."""
+
+    state_floats: int = 0
+
+    def forward(self, ctx, norm: "Norm", x: torch.Tensor, pending, line: LineView, offset: int):
+        """Norms x + pending and returns (the stream with the sum in it, the rows that the mixer reads)."""
+        raise NotImplementedError
+
 
 class Addition(Part):
     """A part behind a layer's block that adds to the stream once more; it may read the step's token ids
@@ -257,11 +292,29 @@ class Block:
         self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
         # norms behind the sublayers, for the arrangements that have them
         self.mixer_out_norm, self.feed_forward_out_norm = mixer_out_norm, feed_forward_out_norm
+        self.mixer_input: Optional[MixerInput] = None
+
+    takes_mixer_input: bool = False      # whether the arrangement has a place for a part in front of the mixer
+
+    def set_mixer_input(self, part: MixerInput) -> None:
+        if not self.takes_mixer_input:
+            raise ValueError(f"{type(self).__name__} has no place for a part between the norm and the mixer")
+        self.mixer_input = part
 
     def parts(self) -> list[Part]:
         """The block's parts; a layer without a feed-forward has neither it nor its norms."""
-        return [part for part in (self.mixer_norm, self.mixer, self.mixer_out_norm, self.feed_forward_norm, self.feed_forward,
-                                  self.feed_forward_out_norm) if part is not None]
+        return [part for part in (self.mixer_norm, self.mixer_input, self.mixer, self.mixer_out_norm, self.feed_forward_norm,
+                                  self.feed_forward, self.feed_forward_out_norm) if part is not None]
+
+    def cache_need(self) -> CacheNeed:
+        """What a run of the block needs of its cache line: the mixer's keys, values and state, and behind that state
+        the one of the part in front of the mixer."""
+        need = self.mixer.cache_need()
+        return need.with_state_behind(self.mixer_input.state_floats) if self.mixer_input is not None else need
+
+    def input_offset(self) -> int:
+        """Where, in a copy of the line's state, the part in front of the mixer has its own."""
+        return self.mixer.cache_need().copy_floats
 
     def forward(self, ctx, x, pending, line: LineView, writes_cache: bool):
         raise NotImplementedError
@@ -269,7 +322,7 @@ class Block:
 
 _REGISTRIES: dict[str, dict[str, Callable[..., Any]]] = {
     "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "block": {}, "embedding": {}, "head": {},
-    "connector": {}, "addition": {},
+    "connector": {}, "addition": {}, "mixer_input": {},
 }
 
 

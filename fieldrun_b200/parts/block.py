@@ -13,10 +13,17 @@ from .norm import LayerNorm
 
 
 class PreNormBlock(Block):
+    """With a part between the norm and the mixer (``mixer_input``), that part runs the norm and gives the mixer's rows."""
+
+    takes_mixer_input = True
+
     def forward(self, ctx, x, pending, line, writes_cache):
         if not self.mixer_norm.accepts_deferred:
             pending = as_tensor(ctx, pending)
-        act, _ = self.mixer_norm.forward(ctx, x, delta=pending)
+        if self.mixer_input is not None:
+            x, act = self.mixer_input.forward(ctx, self.mixer_norm, x, pending, line, self.input_offset())
+        else:
+            act, _ = self.mixer_norm.forward(ctx, x, delta=pending)
         update = self.mixer.forward(ctx, act, line, writes_cache)
         if self.feed_forward is None:                  # a layer without feed-forward: the next norm adds the mixer's update
             return x, update

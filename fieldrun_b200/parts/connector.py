@@ -2,7 +2,9 @@
 
 ``stream_reentry``: x <- W [x ; x0] + step[index], with x0 the embedding's rows, W [width, 2 width] (x's columns
 first) and one vector ``step[index]`` per pass.  A model that runs a stretch of its layers several times with the
-same weights puts this in front of every pass."""
+same weights puts this in front of every pass.
+
+``stream_sum``: x <- x + x0, nothing else and no tensors; the sum is left to the norm that reads the stream next."""
 from __future__ import annotations
 
 from typing import Optional
@@ -11,7 +13,7 @@ import torch
 
 from ..csrc import ops
 from ..weights.loader import MATRIX, VECTOR, TensorNeed, TensorSource
-from .base import Connector, as_tensor, register_part
+from .base import BiasedRows, Connector, UpdateSum, as_tensor, register_part
 from .linear import linear
 
 
@@ -41,4 +43,19 @@ class StreamReentry(Connector):
         return x
 
 
+class StreamSum(Connector):
+    replayable = True
+
+    def forward_deferred(self, ctx, x, pending, first, index):
+        if pending is not None and not isinstance(pending, (torch.Tensor, BiasedRows)):
+            pending = as_tensor(ctx, pending)
+        return x, UpdateSum([pending, first]) if pending is not None else first
+
+    def forward(self, ctx, x, pending, first, index):
+        x, pending = self.forward_deferred(ctx, x, pending, first, index)
+        ops.add_rows(x, as_tensor(ctx, pending))
+        return x
+
+
 register_part("connector", "stream_reentry", StreamReentry, replace=True)
+register_part("connector", "stream_sum", StreamSum, replace=True)

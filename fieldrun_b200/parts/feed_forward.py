@@ -369,7 +369,11 @@ class DenseUnit(FeedForward):
     """W_down act(W_up x): one product in, an activation, one product out.  ``activation`` is one of
     ``ops.ACTIVATIONS`` (``relu_squared``: relu(z)^2, ``gelu_tanh``, ``silu``, ``relu``).  A prompt's rows in bfloat16
     take the first product on tcgen05 with the activation in its epilogue (the step as one expert's rows); few rows,
-    float32 and sizes that kernel does not take go through the plain product and the activation kernel."""
+    float32 and sizes that kernel does not take go through the plain product and the activation kernel.
+
+    ``activation: poly_norm``: act(z) = a N(z) + b N(z^2) + c N(z^3) + e with four learned numbers (a, b, c, e), powers
+    element by element and N(v) = v / sqrt(mean(v^2) + norm_eps) over the row.  It needs the whole row's sums, so it is a
+    kernel of its own behind the plain product."""
 
     replayable = True
     kernel_groups = ("common", "streams", "products")
@@ -379,9 +383,12 @@ class DenseUnit(FeedForward):
         self.hidden_size = int(spec.args["hidden_size"])
         self.width = int(spec.args["width"])
         self.activation = str(spec.args["activation"])
-        if self.activation not in ops.ACTIVATIONS:
-            raise ValueError(f"activation {self.activation!r} is none of {sorted(ops.ACTIVATIONS)}")
-        if not (dtype == torch.bfloat16 and self.width % 128 == 0 and self.hidden_size % 64 == 0):
+        self.normed_powers = self.activation == "poly_norm"
+        self.norm_eps = float(spec.args.get("norm_eps", 1e-6))
+        self.coefficients: Optional[torch.Tensor] = None
+        if self.activation not in ops.ACTIVATIONS and not self.normed_powers:
+            raise ValueError(f"activation {self.activation!r} is none of {sorted(ops.ACTIVATIONS) + ['poly_norm']}")
+        if self.normed_powers or not (dtype == torch.bfloat16 and self.width % 128 == 0 and self.hidden_size % 64 == 0):
             self.kernel_groups = ("common", "streams")         # sizes the tcgen05 product never takes
         self.w_up: Optional[torch.Tensor] = None
         self.w_down: Optional[torch.Tensor] = None
@@ -389,14 +396,18 @@ class DenseUnit(FeedForward):
 
     def _needs(self):
         d, i = self.hidden_size, self.width
-        return (TensorNeed(self.name_of("w_up"), (i, d), MATRIX, "normal"),
-                TensorNeed(self.name_of("w_down"), (d, i), MATRIX, "normal"))
+        needs = [TensorNeed(self.name_of("w_up"), (i, d), MATRIX, "normal"),
+                 TensorNeed(self.name_of("w_down"), (d, i), MATRIX, "normal")]
+        if self.normed_powers:
+            needs.append(TensorNeed(self.name_of("coefficients"), (4,), VECTOR, "around_half"))
+        return needs
 
     def tensor_needs(self):
         return list(self._needs())
 
     def load(self, source: TensorSource) -> None:
-        self.w_up, self.w_down = (source.fetch(n) for n in self._needs())
+        self.w_up, self.w_down, *rest = (source.fetch(n) for n in self._needs())
+        self.coefficients = rest[0] if rest else None
 
     def fused_tiles(self, ctx, rows: int):
         """The lists that make the step one expert's rows in tiles, for the tcgen05 product; they depend on the number
@@ -416,7 +427,9 @@ class DenseUnit(FeedForward):
     def forward(self, ctx, act, act32):
         rows = act.shape[0]
         hidden = ctx.buffer("dense.hidden", (rows, self.width), self.dtype)
-        if (self.dtype == torch.bfloat16 and rows >= FUSED_ACTIVATION_ROWS and not ctx.is_decode and self.width % 128 == 0
+        if self.normed_powers:
+            ops.poly_norm(linear(act, self.w_up), self.coefficients, self.norm_eps, hidden)
+        elif (self.dtype == torch.bfloat16 and rows >= FUSED_ACTIVATION_ROWS and not ctx.is_decode and self.width % 128 == 0
                 and self.hidden_size % 64 == 0):
             # a prompt's rows: product and activation in one kernel on tcgen05, the result rounded once to bfloat16
             tile_expert, tile_row0, num_tiles, offsets, count, tile_rows = self.fused_tiles(ctx, rows)

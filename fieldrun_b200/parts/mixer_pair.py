@@ -60,6 +60,7 @@ class MixerPair(Mixer):
             raise ValueError("a pair of mixers shares one cache line: only one of the two may keep a state")
         kv, st = (a if a.kv_heads else b), (a if a.state_shape else b)
         return CacheNeed(kv_heads=kv.kv_heads, head_dim=kv.head_dim, window=kv.window, value_dim=kv.value_dim, chunk=kv.chunk,
+                         value_heads=kv.value_heads, keep_first=kv.keep_first,
                          state_shape=st.state_shape, state_dtype=st.state_dtype)
 
     def prepare(self, num_positions: int, device) -> None:

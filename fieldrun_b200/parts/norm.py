@@ -13,7 +13,7 @@ import torch
 
 from ..csrc import ops
 from ..weights.loader import VECTOR, TensorNeed, TensorSource
-from .base import Norm, NormedUpdate, UpdateSum, WeightedPair, WeightedRows, as_tensor, register_part
+from .base import BiasedRows, Norm, NormedUpdate, UpdateSum, WeightedPair, WeightedRows, as_tensor, register_part
 
 # FIELDRUN_B200_FUSED_OUTPUT_NORM=0: an update with a norm of its own is normed and added by kernels of their own first
 FUSED_OUTPUT_NORM = os.environ.get("FIELDRUN_B200_FUSED_OUTPUT_NORM", "1") != "0"
@@ -45,7 +45,8 @@ class RMSNorm(Norm):
             return inner.a, inner.b, inner.wa, inner.wb, None
         if isinstance(inner, WeightedRows) and inner.top_k <= ops.NORM_MAX_SUMMED_ROWS:
             return None, None, 1.0, 1.0, (inner.rows, inner.weights, inner.row_map)
-        if isinstance(inner, UpdateSum) and len(inner.tensors) <= 2 and all(w.top_k <= ops.NORM_MAX_SUMMED_ROWS for w in inner.weighted):
+        if (isinstance(inner, UpdateSum) and inner.vector is None and len(inner.tensors) <= 2
+                and all(w.top_k <= ops.NORM_MAX_SUMMED_ROWS for w in inner.weighted)):
             tensors = list(inner.tensors) + [None, None]
             weighted = inner.weighted[0] if inner.weighted else None
             return tensors[0], tensors[1], 1.0, 1.0, (weighted.rows, weighted.weights, weighted.row_map) if weighted else None
@@ -154,7 +155,8 @@ class LayerNorm(Norm):
 class DynamicTanh(Norm):
     """tanh(alpha v) * weight + bias with one learned scalar alpha: a norm without statistics.  Two of them that read
     the same stream (a block whose sublayers run side by side) go through one kernel (``forward_pair``), which also
-    adds the updates that the block before left: float32 tensors and the experts' weighted rows."""
+    adds the updates that the block before left: float32 tensors and the experts' weighted rows.  ``forward_shifted``:
+    norm, updates and a token shift behind the norm in one pass."""
 
     replayable = True
     accepts_deferred = True
@@ -180,25 +182,31 @@ class DynamicTanh(Norm):
 
     @staticmethod
     def split(ctx, delta):
-        """(float32 tensors, experts' rows or None) of whatever form the update came in."""
+        """(float32 tensors, experts' rows or None, a vector for every row or None) of whatever form the update came in."""
         if delta is None:
-            return (), None
+            return (), None, None
         if isinstance(delta, torch.Tensor):
-            return (delta,), None
+            return (delta,), None, None
+        if isinstance(delta, BiasedRows):
+            return (delta.rows,), None, delta.vector
         if isinstance(delta, WeightedRows) and delta.top_k <= ops.NORM_MAX_SUMMED_ROWS:
-            return (), (delta.rows, delta.weights, delta.row_map)
-        if isinstance(delta, UpdateSum) and len(delta.tensors) <= 2 and all(
+            return (), (delta.rows, delta.weights, delta.row_map), None
+        if isinstance(delta, UpdateSum) and len(delta.tensors) <= 2 and not (delta.weighted and delta.vector is not None) and all(
                 w.top_k <= ops.NORM_MAX_SUMMED_ROWS for w in delta.weighted):
             weighted = delta.weighted[0] if delta.weighted else None
-            return tuple(delta.tensors), (weighted.rows, weighted.weights, weighted.row_map) if weighted else None
-        return (as_tensor(ctx, delta),), None
+            return (tuple(delta.tensors), (weighted.rows, weighted.weights, weighted.row_map) if weighted else None,
+                    delta.vector)
+        return (as_tensor(ctx, delta),), None, None
 
     def forward(self, ctx, x, *, delta=None, rows=None, want32=False, write_back=True):
-        deltas, experts = self.split(ctx, delta)
+        deltas, experts, vector = self.split(ctx, delta)
         count = rows.numel() if rows is not None else x.shape[0]
         out = ctx.buffer(f"norm.out.{self.width}", (count, self.width), self.dtype)
-        ops.dyt_norm(x, self.triple(), out, deltas=deltas, experts=experts, rows=rows,
-                     write_back=write_back and rows is None and (bool(deltas) or experts is not None))
+        write = write_back and rows is None and (bool(deltas) or experts is not None)
+        if experts is None:
+            ops.dyt_rows(x, self.triple(), out, deltas=deltas, vector=vector, rows=rows, stream=x if write else None)
+        else:
+            ops.dyt_norm(x, self.triple(), out, deltas=deltas, experts=experts, rows=rows, write_back=write)
         out32 = None
         if want32:
             out32 = out
@@ -210,7 +218,9 @@ class DynamicTanh(Norm):
     def forward_pair(self, ctx, x, other: "DynamicTanh", *, delta=None, want32=False):
         """This norm and ``other`` of the same x + delta (the sum stored back): (out, other's out, other's out in
         float32 or None)."""
-        deltas, experts = self.split(ctx, delta)
+        deltas, experts, vector = self.split(ctx, delta)
+        if vector is not None:                                       # the kernel for two norms takes no vector
+            deltas, experts = (as_tensor(ctx, delta),), None
         rows = x.shape[0]
         out1 = ctx.buffer(f"norm.out.{self.width}", (rows, self.width), self.dtype)
         out2 = ctx.buffer(f"norm.out2.{self.width}", (rows, self.width), self.dtype)
@@ -220,6 +230,25 @@ class DynamicTanh(Norm):
         ops.dyt_norm(x, self.triple(), out1, second=other.triple(), out2=out2, out2_32=out2_32, deltas=deltas, experts=experts,
                      write_back=bool(deltas) or experts is not None)
         return out1, out2, (out2 if self.dtype == torch.float32 else out2_32) if want32 else None
+
+
+    def forward_shifted(self, ctx, x, share, line_state, offset, *, delta=None):
+        """h = norm(x + delta), and every row moved towards the one before it: h_t + (h_(t-1) - h_t) * share, the row
+        before a step's first one being state of the sequence (``line_state``, at ``offset``).  Returns (the stream with
+        the sum, the rows).  A row's neighbour is normed again where it is needed, so the sum goes into a second buffer:
+        nobody may overwrite the stream that a neighbour still reads."""
+        deltas, experts, vector = self.split(ctx, delta)
+        if experts is not None:
+            deltas, vector = (as_tensor(ctx, delta),), None
+        rows = x.shape[0]
+        stream = None
+        if deltas:
+            buffers = [ctx.buffer(name, (rows, self.width), torch.float32) for name in ("stream", "stream.other")]
+            stream = next(b for b in buffers if b.data_ptr() != x.data_ptr())
+        out = ctx.buffer(f"norm.out.{self.width}", (rows, self.width), self.dtype)
+        ops.dyt_rows(x, self.triple(), out, deltas=deltas, vector=vector, stream=stream,
+                     shift=(share, ctx, line_state, offset))
+        return x if stream is None else stream, out
 
 
 register_part("norm", "dynamic_tanh", DynamicTanh, replace=True)

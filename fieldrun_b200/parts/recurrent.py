@@ -1,4 +1,4 @@
-"""Mixers that carry a float32 state from token to token instead of keys and values, each behind a short causal
+"""Mixers that carry a float32 state from token to token instead of keys and values, most of them behind a short causal
 convolution whose last inputs are part of the state too (kernels: scans.cu).
 
 ``selective_scan`` (Mamba): [x | z] = W_in h; x <- silu(conv(x)); [dt | B | C] = W_x x; dt <- softplus(W_dt dt + b);
@@ -15,6 +15,8 @@ convolution whose last inputs are part of the state too (kernels: scans.cu).
     sigmoid(W_b h), g = exp(-exp(A_log_h) softplus(W_a h + dt_bias_h)), one of each per head; per head (head h uses q/k
     head h // (heads / kv_heads)):  S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q (S is [head_dim, value_dim]);
     o / rms(o) * w (w [value_dim], shared by the heads) * silu(W_g h), then W_o.  Kernel: delta_rule.cu.
+``min_gru`` (no convolution): z = sigmoid(W_z h + b_z), u = W_x h + b_x; the candidate is u + 1/2 where u >= 0 and sigmoid(u)
+    where u < 0;  S <- (1 - z) S + z candidate, element by element;  out = W_o (S * silu(W_g h)).
 
 The state of a slot lies in the cache line's state area as [2, floats] float32 (two copies, see scans.cu): the
 recurrence's state first, the convolution's last inputs behind it.  The projections are library products with
@@ -284,6 +286,47 @@ class GatedDeltaRule(_StateMixer):
         return linear(out, w["o_proj"])
 
 
+class MinGru(_StateMixer):
+    def __init__(self, spec, dtype):
+        super().__init__(spec, dtype)
+        a = spec.args
+        self.hidden_size, self.width = int(a["hidden_size"]), int(a["width"])
+        if self.width < 1:
+            raise ValueError(f"a gated recurrence of width {self.width}")
+        self.state_floats = self.width
+        # columns of the one product in: z | x | gate, then zero rows up to a multiple of 16
+        self.in_rows = -(-3 * self.width // 16) * 16
+        self.w_in: Optional[torch.Tensor] = None
+        self.w: dict[str, torch.Tensor] = {}
+
+    def _needs(self) -> dict[str, TensorNeed]:
+        d, c = self.hidden_size, self.width
+        return {
+            "z_proj": TensorNeed(self.name_of("z_proj"), (c, d), MATRIX, "normal"),
+            "z_bias": TensorNeed(self.name_of("z_bias"), (c,), VECTOR, "bias"),
+            "x_proj": TensorNeed(self.name_of("x_proj"), (c, d), MATRIX, "normal"),
+            "x_bias": TensorNeed(self.name_of("x_bias"), (c,), VECTOR, "bias"),
+            "gate_proj": TensorNeed(self.name_of("gate_proj"), (c, d), MATRIX, "normal"),
+            "o_proj": TensorNeed(self.name_of("o_proj"), (d, c), MATRIX, "normal"),
+        }
+
+    def load(self, source: TensorSource) -> None:
+        w = self._fetch(source)
+        stacked = [w.pop(n) for n in ("z_proj", "x_proj", "gate_proj")]
+        self.w_in = torch.zeros((self.in_rows, self.hidden_size), dtype=stacked[0].dtype, device=stacked[0].device)
+        torch.cat(stacked, dim=0, out=self.w_in[:3 * self.width])
+        self.w = w
+
+    def forward(self, ctx, act: torch.Tensor, line: LineView, writes_cache: bool) -> torch.Tensor:
+        self._check(writes_cache)
+        w, rows, c = self.w, act.shape[0], self.width
+        proj = linear(act, self.w_in)                                            # float32 [T, in_rows]: z | x | gate, before biases
+        out = ctx.buffer("min_gru.y", (rows, c), self.dtype)
+        ops.min_gru(proj, 0, c, 2 * c, w["z_bias"], w["x_bias"], ctx, line.state, 0, out)
+        return linear(out, w["o_proj"])
+
+
+register_part("mixer", "min_gru", MinGru, replace=True)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule, replace=True)
 register_part("mixer", "selective_scan", SelectiveScan, replace=True)
 register_part("mixer", "gated_linear_recurrence", GatedLinearRecurrence, replace=True)
