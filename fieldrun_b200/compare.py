@@ -21,6 +21,10 @@ clamped gate fed with weighted inputs) beside a MiniMax-M2 model with as many ex
 a sink, then twice capped attention beside a gated delta rule, in turn; experts chosen among the best groups plus a
 gated shared expert) beside a MiniMax-M2 model with as many experts of the same size.
 
+``--design duzinex``: a Duzinex model (differential attention, retention, differential attention and a gated recurrence in
+turn, each behind a token shift; a feed-forward of normed powers) beside a Bamasun and a MiniMax-M2 model of equal width,
+projections and feed-forward weights.
+
 The weights of every model are far larger than the L2 cache, and each timed step reads all of them.
 """
 from __future__ import annotations
@@ -137,6 +141,29 @@ def bakasun_config(width, heads, kv_heads, dim, ff, layers, vocab) -> dict[str, 
     return {"architecture": "Bakasun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": listed}
 
 
+# the Duzinex comparison: a head's two maps of half the head size each, over values of the whole one, make projections and cache
+# lines of the sizes that plain attention has; the first four tokens stay visible beside the window
+DUZINEX_WINDOW, DUZINEX_KEEP = 1024, 4
+
+
+def duzinex_config(width, heads, kv_heads, dim, ff, layers, vocab) -> dict[str, Any]:
+    """Layers in turns of four: attention, retention (heads of ``dim`` x ``dim``), attention, gated recurrence."""
+    mlp = {"kind": "dense", "ff": ff}
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim // 2, "vdim": dim, "scale": (dim // 2) ** -0.5, "diff": 0.5, "softcap": 30.0,
+             "mask": {"size": DUZINEX_WINDOW, "keep_first": DUZINEX_KEEP}, "rot": {"base": 500000.0, "dims": dim // 2}}
+    decay = [1.0 - 2.0 ** (-5.0 - 7.0 * h / max(heads - 1, 1)) for h in range(heads)]
+    listed = []
+    for index in range(layers):
+        turn = index % 4
+        if turn == 1:
+            listed.append({"type": "retention", "mixer": {"heads": heads, "dim": dim, "vdim": dim, "decay": decay}, "mlp": mlp})
+        elif turn == 3:
+            listed.append({"type": "mingru", "mixer": {"width": width}, "mlp": mlp})
+        else:
+            listed.append({"type": "attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Duzinex", "vocab": vocab, "width": width, "embedding": {"scale": 8.0}, "norm": {"eps": 1e-6}, "layers": listed}
+
+
 def minimax_config(width, heads, kv_heads, dim, ff, layers, vocab, experts=None) -> dict[str, Any]:
     if experts is not None:
         count, top, expert_ff = experts
@@ -236,6 +263,8 @@ def compare_designs(sizes=("w2048", "w4096"), steps: int = 8, warmup: int = 3, d
         elif design == "depelix":
             experts = (DEPELIX_EXPERTS, DEPELIX_TOP, size["ff"] // DEPELIX_FF_SHARE // 128 * 128)
             pair = (("depelix", depelix_config(**size)), ("minimax_m2", minimax_config(**size, experts=experts)))
+        elif design == "duzinex":
+            pair = (("duzinex", duzinex_config(**size)), ("bamasun", bamasun_config(**size)), ("minimax_m2", minimax_config(**size)))
         else:
             pair = (("bamasun", bamasun_config(**size)), ("minimax_m2", minimax_config(**size)))
         for design_name, config in pair:

@@ -67,7 +67,7 @@ _SIGNATURES = {
     "frb_map_difference": "pppi" "iiiiff",
     "frb_poly_norm": "pppiiif",
     "frb_min_gru": "piiii" "pp" "ppp" "pll" "pi" "iii",
-    "frb_retention": "piiiii" "pppp" "pll" "pip" "iiiii" "ff",
+    "frb_retention": "piiiiii" "pppp" "pll" "pip" "iiiii" "ff",
     "frb_embed_pair_rows": "pppipiiifillppppppi",
     "frb_token_side_gate": "pppipiiiiii",
     "frb_add_rms_normed": "pppiif",
@@ -484,6 +484,11 @@ def retention_takes(dim: int, vdim: int) -> bool:
     return 1 <= dim <= 1024 and vdim >= 1
 
 
+def retention_chunks_take(dim: int, vdim: int) -> bool:
+    """Whether a bfloat16 prompt of heads with these sizes goes chunk by chunk on tensor cores."""
+    return dim % 8 == 0 and dim <= 128 and vdim % 8 == 0
+
+
 def retention_decays(values, device) -> torch.Tensor:
     """float32 [heads, 2, RETENTION_CHUNK + 1]: decay^n and decay^n - 1 for n = 0, 1, ..., made in float64, rounded once."""
     d = torch.tensor([float(v) for v in values], dtype=torch.float64)[:, None]
@@ -494,14 +499,15 @@ def retention_decays(values, device) -> torch.Tensor:
 
 def retention(proj: torch.Tensor, offsets: tuple[int, int, int, int], decays: torch.Tensor, ctx, state: torch.Tensor, state_offset: int,
               out: torch.Tensor, raw: torch.Tensor, *, heads: int, dim: int, vdim: int, k_scale: float, eps: float) -> None:
-    """Per head S <- decay S + (k_scale k) v^T, o = S^T q, out = o / sqrt(mean(o^2) + eps) * silu(g): q, k, v, g in float32
-    columns of ``proj`` at the four ``offsets``; ``decays`` as :func:`retention_decays` makes them; ``raw``: float32 scratch of
-    the outputs' size."""
-    for t in (proj, decays, raw):
+    """Per head S <- decay S + (k_scale k) v^T, o = S^T q, out = o / sqrt(mean(o^2) + eps) * silu(g): q, k, v, g in columns of
+    ``proj`` at the four ``offsets``; ``decays`` as :func:`retention_decays` makes them; ``raw``: float32 scratch of the outputs'
+    size.  ``proj`` in float32: token by token; in bfloat16 (sizes for which :func:`retention_chunks_take` holds): chunk by chunk
+    on tensor cores."""
+    for t in (decays, raw):
         _want(t, torch.float32, "retention's inputs")
     if raw.numel() < out.numel() or decays.shape[0] != heads or decays.shape[-1] != RETENTION_CHUNK + 1:
         raise KernelError("retention: the scratch is smaller than the outputs, or the decays are not the heads'")
-    _call("frb_retention", _ptr(proj), proj.shape[1], *(int(o) for o in offsets), _ptr(decays), _ptr(ctx.seq_slot), _ptr(ctx.seq_start),
+    _call("frb_retention", _ptr(proj), _code(proj.dtype), proj.shape[1], *(int(o) for o in offsets), _ptr(decays), _ptr(ctx.seq_slot), _ptr(ctx.seq_start),
           _ptr(ctx.cu_q_len), *_state_place(state, state_offset), _ptr(out), _code(out.dtype), _ptr(raw), proj.shape[0], ctx.num_seqs,
           int(heads), int(dim), int(vdim), float(k_scale), float(eps))
 

@@ -15,7 +15,7 @@ import torch
 from ..cache import CacheNeed, SequenceCache
 from ..config.plan import ModelPlan
 from ..parts import build_block, build_part
-from ..parts.linear import require_true_float32
+from ..parts.linear import full_sums, require_true_float32
 from ..weights.loader import TensorNeed, TensorSource
 from .context import StepContext
 
@@ -91,6 +91,7 @@ class DecoderModel:
     def load(self, source: TensorSource) -> None:
         if self.dtype == torch.float32:
             require_true_float32()
+        full_sums()
         self.embedding.load(source)
         for connector in self.connectors:
             connector.load(source)

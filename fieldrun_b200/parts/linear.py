@@ -42,8 +42,20 @@ def require_true_float32() -> None:
         torch.backends.cuda.matmul.allow_fp16_reduced_precision_reduction = False
 
 
-def linear(rows: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """rows [T, in] @ weight[out, in]^T -> float32 [T, out]."""
+def full_sums() -> None:
+    """Products with a bfloat16 result add in float32 to the end and round once."""
+    if hasattr(torch.backends.cuda.matmul, "allow_bf16_reduced_precision_reduction"):
+        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+
+
+def linear(rows: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None, rounded: bool = False) -> torch.Tensor:
+    """rows [T, in] @ weight[out, in]^T -> float32 [T, out]; with ``rounded`` (bfloat16 rows only) the float32 sums rounded once
+    to bfloat16, for a reader that takes its operands in that type anyway."""
+    if rounded:
+        if rows.dtype != torch.bfloat16 or weight.dtype != torch.bfloat16 or not rows.is_cuda or out is not None:
+            raise RuntimeError(f"a rounded matrix product of {rows.dtype} rows with a {weight.dtype} weight on {rows.device}")
+        with ops.timed(f"library_mm_bf16[{weight.shape[0]}x{weight.shape[1]}]"):
+            return torch.mm(rows, weight.t())
     if not rows.is_cuda:
         raise RuntimeError("fieldrun_b200 runs on a CUDA device only; a CPU tensor reached a matrix product")
     if rows.dtype != weight.dtype:

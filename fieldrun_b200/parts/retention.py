@@ -25,6 +25,8 @@ from ..weights.loader import MATRIX, TensorNeed, TensorSource
 from .base import Mixer, register_part
 from .linear import linear
 
+CHUNK_MIN_TOKENS = 8           # steps whose longest run of new tokens is shorter go token by token
+
 
 class Retention(Mixer):
     replayable = True
@@ -85,7 +87,9 @@ class Retention(Mixer):
         if not writes_cache:
             raise ValueError("a recurrent layer cannot read another layer's state: it has to write its own")
         rows = act.shape[0]
-        proj = linear(act, self.w_in)                                       # float32 [T, in_rows]: q | k | v | gate
+        # q | k | v | gate: float32 for the recurrence token by token; a bfloat16 prompt's chunks take them in bfloat16
+        chunks = self.dtype == torch.bfloat16 and ctx.max_q_len >= CHUNK_MIN_TOKENS and ops.retention_chunks_take(self.head_dim, self.value_dim)
+        proj = linear(act, self.w_in, rounded=chunks)                       # [T, in_rows]
         out = ctx.buffer("retention.out", (rows, self.v_width), self.dtype)
         raw = ctx.buffer("retention.raw", (rows, self.v_width), torch.float32)      # for steps that cut the heads over blocks
         ops.retention(proj, self.offsets, self.decay, ctx, line.state, 0, out, raw, heads=self.num_heads, dim=self.head_dim,

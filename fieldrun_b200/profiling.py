@@ -536,7 +536,53 @@ def output_norm(launches: int, tokens: int) -> dict:
     return result
 
 
+def duzinex(kind: str, launches: int) -> dict:
+    """Kernels of the Duzinex design alone at a width of 2048, over four prompts of 2,048 tokens or 64 single tokens:
+    ``retention`` (16 heads of 128 x 128), ``gru`` (the gated recurrence, 2,048 channels), ``shift`` (norm, residual sum and token
+    shift), ``powers`` (the activation, rows of 8,192)."""
+    name, shape = kind.rsplit("_", 1)
+    lengths = [2048] * 4 if shape == "prefill" else [1] * 64
+    tokens, width = sum(lengths), 2048
+    tables = _Tables(lengths)
+    tables.max_q_len = max(lengths)
+    typed = torch.empty(tokens, width, dtype=torch.bfloat16, device=DEV)
+    state_bytes = 0
+    if name == "retention":
+        heads, dim = 16, 128
+        proj = torch.randn(tokens, 4 * width, device=DEV, dtype=torch.bfloat16 if shape == "prefill" else torch.float32)
+        state = torch.zeros(len(lengths), 2, heads * dim * dim, device=DEV)
+        decays = ops.retention_decays([1.0 - 2.0 ** -(5 + h / 2) for h in range(heads)], DEV)
+        raw = torch.empty(tokens, width, device=DEV)
+        launch = lambda: ops.retention(proj, (0, width, 2 * width, 3 * width), decays, tables, state, 0, typed, raw, heads=heads, dim=dim,
+                                       vdim=dim, k_scale=dim ** -0.5, eps=1e-6)
+        moved, state_bytes = proj.numel() * proj.element_size() + typed.numel() * 2, 2 * state[:, 0].numel() * 4
+    elif name == "gru":
+        proj = torch.randn(tokens, 3 * width, device=DEV)
+        state = torch.zeros(len(lengths), 2, width, device=DEV)
+        bias = torch.zeros(width, device=DEV)
+        launch = lambda: ops.min_gru(proj, 0, width, 2 * width, bias, bias, tables, state, 0, typed)
+        moved = proj.numel() * 4 + typed.numel() * 2
+    elif name == "shift":
+        x, d, stream = (torch.randn(tokens, width, device=DEV) for _ in range(3))
+        w = torch.ones(width, device=DEV)
+        state = torch.zeros(len(lengths), 2, width, device=DEV)
+        launch = lambda: ops.dyt_rows(x, (w, w, w[:1]), typed, deltas=(d,), stream=stream, shift=(w, tables, state, 0))
+        moved = 3 * x.numel() * 4 + typed.numel() * 2
+    elif name == "powers":
+        z, act = torch.randn(tokens, 4 * width, device=DEV), torch.ones(4, device=DEV)
+        typed = torch.empty(tokens, 4 * width, dtype=torch.bfloat16, device=DEV)
+        launch = lambda: ops.poly_norm(z, act, 1e-6, typed)
+        moved = z.numel() * 4 + typed.numel() * 2
+    else:
+        raise ValueError(kind)
+    ms = _time(launch, launches) if shape == "prefill" else _time_recorded(launch, max(launches, 20))
+    return {"case": kind, "tokens": tokens, "ms": round(ms, 4), "gbs": round((moved + state_bytes) / ms / 1e6, 1)}
+
+
 CASES = {
+    **{f"duzinex_{kind}": (lambda n, kind=kind: duzinex(kind, n))
+       for kind in ("retention_prefill", "retention_decode", "gru_prefill", "gru_decode", "shift_prefill", "shift_decode",
+                    "powers_prefill", "powers_decode")},
     "delta_rule_prefill": lambda n: delta_rule("prefill", n),
     "delta_rule_prefill_whole": lambda n: delta_rule("prefill_whole", n),
     "delta_rule_decode": lambda n: delta_rule("decode", n),

@@ -257,7 +257,10 @@ def run_retention(proj, heads, dim, vdim, decay, eps, ctx, state, offset, dtype)
     qk, v = heads * dim, heads * vdim
     out = torch.empty((proj.shape[0], v), dtype=TORCH[dtype], device=DEV)
     raw = torch.full((proj.shape[0], v), float("nan"), device=DEV)
-    ops().retention(f32(proj), (0, qk, 2 * qk, 2 * qk + v), ops().retention_decays(decay, DEV), ctx, state, offset, out, raw, heads=heads,
+    chunks = dtype == "bfloat16" and ctx.max_q_len >= 2 and ops().retention_chunks_take(dim, vdim)
+    if chunks:                                               # rows on 16 bytes, as the part lays them out
+        proj = np.concatenate([proj, np.zeros((proj.shape[0], -proj.shape[1] % 16))], axis=1)
+    ops().retention(dev(proj, torch.bfloat16) if chunks else f32(proj), (0, qk, 2 * qk, 2 * qk + v), ops().retention_decays(decay, DEV), ctx, state, offset, out, raw, heads=heads,
                     dim=dim, vdim=vdim, k_scale=dim ** -0.5, eps=eps)
     return f64(out)
 
