@@ -22,56 +22,17 @@
 //
 // Every wait on an mbarrier gives up after about a second (at once when another wait of the block has given
 // up), sets `status`, and the block leaves through the common exit, which frees the tensor memory.
-#include "tcgen05.cuh"
+#include "attention_tc.cuh"
 
-#define AT_QUERIES 128
 #define AT_THREADS 320         // warp 0: TMA producer, warp 1: MMA issuer and tensor-memory owner, warps 2-9: softmax
 #define AT_SOFTMAX_THREADS 256 // warps 2-5 take the first page of every step, warps 6-9 the second
 #define AT_STAGES 3
 #define AT_STEP_PAGES 2        // cache pages per step of the inner loop
 #define AT_STEP_KEYS (AT_STEP_PAGES * FRB_PAGE)
-#define AT_RAISE 8.0f          // the running maximum follows a page's maximum only beyond this margin
 
 using namespace frb_tma;
 using namespace frb_tc;
-
-namespace {
-
-// 2^x by the special-function unit (relative error about 2^-22; -inf and anything below -126 give 0)
-__device__ __forceinline__ float exp2_fast(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
-// the largest of three (one instruction on this architecture)
-__device__ __forceinline__ float max3(float a, float b, float c) {
-    float d;
-    asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-    return d;
-}
-
-// the hardware's instructions on two float32 values in one 64-bit register
-__device__ __forceinline__ uint64_t pair_of(float lo, float hi) {
-    uint64_t r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
-    return r;
-}
-__device__ __forceinline__ void halves_of(uint64_t v, float& lo, float& hi) {
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-}
-__device__ __forceinline__ uint64_t fma_pairs(uint64_t a, uint64_t b, uint64_t c) {
-    uint64_t d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ uint64_t add_pairs(uint64_t a, uint64_t b) {
-    uint64_t d;
-    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
-
-}  // namespace
+using namespace frb_at;
 
 struct AttnTcParams {
     const int* page_table;
@@ -89,7 +50,7 @@ struct AttnTcParams {
     const float* slopes;       // SLOPED kernels: one slope per query head; key j's score is lowered by slope * (i - j)
     int chunk;                 // 0, or a query sees only the keys of its own chunk of this many positions
     const float* sinks;        // null, or one number per query head whose exponential joins the softmax's denominator
-    float cap_scale, cap2;     // CAPPED kernels (capped_score2): scale / cap and cap * log2(e)
+    float cap_scale, cap2;     // CAPPED kernels (cap_scores): scale / cap and cap * log2(e)
     int keep_first, v_heads;   // first tokens that stay visible beside the window; value heads (runs of key heads share one)
 };
 
@@ -251,15 +212,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
             for (int c = 0; c < FRB_PAGE / 16; ++c) tmem_ld16(mine + 16 * c, raw[c]);
             tmem_wait_ld();
-            // CAPPED: every score becomes cap * tanh(score * scale / cap) * log2(e) first; what follows then sees a scale of one
-            const float scale2 = CAPPED ? 1.f : p.scale2;
-            if (CAPPED) {
-#pragma unroll
-                for (int c = 0; c < FRB_PAGE / 16; ++c)
-#pragma unroll
-                    for (int i = 0; i < 16; ++i)
-                        raw[c][i] = __float_as_uint(capped_score2(__uint_as_float(raw[c][i]), p.cap_scale, p.cap2));
-            }
+            // CAPPED: every score becomes tanh(score * scale / cap) first; what follows then sees a scale of cap * log2(e)
+            const float scale2 = CAPPED ? p.cap2 : p.scale2;
+            if (CAPPED) cap_scores(raw, p.cap_scale);
             // Most pages lie wholly before the tile's first query (and inside the window): no key of theirs is
             // masked for any row of this warp, and the per-key comparisons are left out.
             const bool open_page = __all_sync(0xffffffffu, valid && key0 + FRB_PAGE - 1 <= hi && (key0 >= lo || key0 + FRB_PAGE <= p.keep_first));

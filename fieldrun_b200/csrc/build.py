@@ -31,7 +31,7 @@ class BuildError(RuntimeError):
 GROUPS: dict[str, tuple[str, ...]] = {
     "common": ("elementwise.cu", "layernorm.cu", "attention_generic.cu", "sampling.cu", "stream_ops.cu", "token_inputs.cu",
                "sandwich_norm.cu", "poly_norm.cu"),
-    "attention": ("attention_mma.cu", "attention_decode_tma.cu", "attention_tc.cu"),
+    "attention": ("attention_mma.cu", "attention_decode_tma.cu", "attention_tc.cu", "attention_pair_tc.cu"),
     "streams": ("experts_stream.cu", "experts_mma.cu"),
     "experts": ("routing.cu", "experts_generic.cu"),
     "products": ("experts_tc.cu",),

@@ -63,6 +63,7 @@ _SIGNATURES = {
     "frb_expert_gemm_tc": "pipippppiipiiipif",
     "frb_gather_rows_bf16": "pppii",
     "frb_attention_prefill_tc": "pippipippipppppiiifippipf" "iiii",
+    "frb_attention_pair_tc": "pippi" "pippi" "ppppp" "iiiifiif" "pffp",
     "frb_dyt_rows": "ppppp" "ppp" "pp" "iii" "p" "pppp" "pll",
     "frb_map_difference": "pppi" "iiiiff",
     "frb_poly_norm": "pppiiif",
@@ -96,7 +97,8 @@ _ENTRY_GROUPS = {
                "frb_dyt_rows", "frb_map_difference", "frb_poly_norm"),
     "latent": ("frb_latent_prepare", "frb_latent_queries", "frb_latent_attention", "frb_latent_gate",
                "frb_latent_attention_mma", "frb_latent_attention_tc"),
-    "attention": ("frb_attention_decode_mma", "frb_attention_prefill_mma", "frb_attention_decode_tma", "frb_attention_prefill_tc"),
+    "attention": ("frb_attention_decode_mma", "frb_attention_prefill_mma", "frb_attention_decode_tma", "frb_attention_prefill_tc",
+                  "frb_attention_pair_tc"),
     "streams": ("frb_weight_stream", "frb_expert_gemm_mma"),
     "experts": ("frb_router_topk", "frb_expert_plan", "frb_expert_combine", "frb_expert_gemm_generic", "frb_route_plan_small",
                 "frb_router_small", "frb_router_logits", "frb_scaled_rows"),
@@ -1178,6 +1180,12 @@ _WAIT_CODES = {
     16: "prompt attention: the softmax waiting for the scores",
     18: "prompt attention: the correction waiting for the step before",
     19: "prompt attention: the epilogue waiting for the last steps",
+    31: "attention of two maps: the producer waiting for a free key/value stage",
+    32: "attention of two maps: the query tiles' copies",
+    33: "attention of two maps: the MMA thread waiting for a loaded key/value stage",
+    35: "attention of two maps: the MMA thread waiting for the probabilities",
+    36: "attention of two maps: the softmax waiting for the scores",
+    39: "attention of two maps: the epilogue waiting for the last steps",
     21: "latent attention: the producer waiting for the scores of the page before",
     22: "latent attention: the producer waiting for the sums of the page before",
     23: "latent attention: the MMA thread waiting for the queries",
@@ -1282,6 +1290,27 @@ def attention_prefill_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
           _ptr(seq_q_len), _ptr(cu_q_len), _ptr(out), num_heads, num_kv_heads, head_dim, float(scale), int(window or 0),
           _ptr(tc_status(q.device)), _ptr(slopes), int(chunk or 0), _ptr(sinks), float(softcap or 0.0), int(v_dim or head_dim),
           int(keep_first or 0), num_kv_heads // maps, _maps_output(out))
+
+
+def attention_pair_takes(head_dim: int, v_dim: int) -> bool:
+    """Whether :func:`attention_pair_tc` takes heads of these sizes."""
+    return head_dim == 64 and v_dim in (64, 128)
+
+
+def attention_pair_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, page_table: torch.Tensor, tile_seq: torch.Tensor,
+                      tile_q0: torch.Tensor, seq_slot: torch.Tensor, seq_start: torch.Tensor, seq_q_len: torch.Tensor,
+                      cu_q_len: torch.Tensor, out: torch.Tensor, *, heads: int, v_heads: int, head_dim: int, v_dim: int, scale: float,
+                      window: Optional[int], keep_first: int, softcap: Optional[float], lam: torch.Tensor, eps: float, factor: float) -> None:
+    """Many tokens per sequence on tcgen05, two maps per head over shared values, their difference and its norm in one kernel
+    (what :func:`attention_prefill_tc` with ``maps`` 2 and :func:`map_difference` make in two): tiles of 128 queries of one head,
+    ``out`` [T, heads * v_dim] in bfloat16."""
+    for t in (q, k_pages, v_pages, out):
+        _want(t, torch.bfloat16, "tensor-core attention operands")
+    _want(lam, torch.float32, "lambda")
+    _call("frb_attention_pair_tc", _ptr(q), q.shape[0], _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(page_table),
+          page_table.shape[1], _ptr(tile_seq), _ptr(tile_q0), tile_seq.numel(), _ptr(seq_slot), _ptr(seq_start), _ptr(seq_q_len),
+          _ptr(cu_q_len), _ptr(out), int(heads), int(v_heads), int(head_dim), int(v_dim), float(scale), int(window or 0),
+          int(keep_first or 0), float(softcap or 0.0), _ptr(lam), float(eps), float(factor), _ptr(tc_status(q.device)))
 
 
 def wait_probe(device, limit_cycles: int = 100_000) -> int:

@@ -32,8 +32,8 @@ each an attention of its own with queries and keys of ``head_dim`` over the same
 
 A projection's rows are laid out head by head as [map 1, map 2]; the kernels see the two maps as query heads and key heads of
 their own (rows are put into the order key head, map, query head of the group at load), two key heads sharing a value head.
-The difference is taken in float32: of the one-token kernels' partial results where those are joined, of float32 outputs
-otherwise.
+The difference is taken in float32: of the one-token kernels' partial results where those are joined, inside the kernel that
+runs both maps of a prompt's head, of float32 outputs otherwise.
 """
 from __future__ import annotations
 
@@ -262,6 +262,13 @@ class GQAAttention(Mixer):
             elif self.head_dim in ops.TC_ATTENTION_HEAD_DIMS and ctx.max_q_len >= TC_ATTENTION_MIN_QUERIES:
                 # prompts: 128 queries of one head per block, both products on tcgen05
                 tile_seq, tile_q0 = ctx.query_tiles(ops.TC_ATTENTION_QUERIES)
+                if self.maps == 2 and self.chunk is None and ops.attention_pair_takes(self.head_dim, self.value_dim):
+                    # both maps, their difference and its norm in one kernel
+                    ops.attention_pair_tc(q, line.keys, line.values, line.page_table, tile_seq, tile_q0, ctx.seq_slot, ctx.seq_start,
+                                          ctx.seq_q_len, ctx.cu_q_len, out, heads=self.num_heads, v_heads=self.num_kv_heads,
+                                          head_dim=self.head_dim, v_dim=self.value_dim, scale=self.softmax_scale, window=self.window,
+                                          keep_first=self.keep_first, softcap=self.softcap, **difference)
+                    return
                 ops.attention_prefill_tc(q, line.keys, line.values, line.page_table, tile_seq, tile_q0, ctx.seq_slot,
                                          ctx.seq_start, ctx.seq_q_len, ctx.cu_q_len, maps_out, **common)
             else:

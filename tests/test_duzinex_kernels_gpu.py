@@ -486,6 +486,14 @@ def test_many_token_kernels_leave_two_maps_in_float32(heads, kv_heads, dim, vdim
                            dev(np.array([s for s, _ in seqs], dtype=np.int32)), dev(q_lens), dev(cu), maps, **c["args"])
     ops().tc_status_check(DEV)
     close(f64(maps), c["maps"], 1.2e-2, kernel)
+    if kernel == "attention_prefill_tc" and ops().attention_pair_takes(dim, vdim):
+        # both maps, their difference and its norm in one kernel
+        out = torch.full((len(c["rows"]), heads * vdim), 7.0, dtype=torch.bfloat16, device=DEV)
+        ops().attention_pair_tc(c["q"], c["kc"], c["vc"], c["table"], dev(tile_seq), dev(tile_q0), dev(np.arange(len(seqs), dtype=np.int32)),
+                                dev(np.array([s for s, _ in seqs], dtype=np.int32)), dev(q_lens), dev(cu), out, heads=heads, v_heads=kv_heads,
+                                head_dim=dim, v_dim=vdim, scale=SCALE, window=window, keep_first=keep, softcap=softcap, **c["difference"])
+        ops().tc_status_check(DEV)
+        close(f64(out), c["want"], 2.5e-2, "one kernel")
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
