@@ -162,9 +162,13 @@ attention_pair_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         const bool valid = q0 + row < q_len;
         const int hi = valid ? start + q0 + row : -1;
         const int lo = valid ? first_visible_key(hi, p.window, 0) : 0;
-        const float scale2 = CAPPED ? p.cap2 : p.scale2;
+        const float scale2 = CAPPED ? 1.f : p.scale2;
         float m_used = -INFINITY, l_sum = 0.f;
         bool ok = true;
+        // whether every key of a page is visible to every row of the warp: most pages are, and need no comparisons
+        auto open_page = [&](int key0) {
+            return __all_sync(0xffffffffu, valid && key0 + FRB_PAGE - 1 <= hi && (key0 >= lo || key0 + FRB_PAGE <= p.keep_first));
+        };
         for (int j = 0; j < num_steps; ++j) {
             // a wait that gives up does not end the loop: the block's later waits then return at once
             if (!bar_wait(&s_full[m], j & 1, failed)) { if (ok && lane == 0) atomicExch(p.status, 36); ok = false; }
@@ -172,18 +176,14 @@ attention_pair_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             const int pages = min(AP_STEP_PAGES, num_pages - AP_STEP_PAGES * j);
             // the step's largest visible score, before its cap (which keeps the order)
             float step_max = -INFINITY;
-            int key0[AP_STEP_PAGES];
-            bool open[AP_STEP_PAGES];
-#pragma unroll
-            for (int h = 0; h < AP_STEP_PAGES; ++h) {
-                if (h >= pages) break;
-                key0[h] = run_at(AP_STEP_PAGES * j + h, kept, first_page) * FRB_PAGE;
-                open[h] = __all_sync(0xffffffffu, valid && key0[h] + FRB_PAGE - 1 <= hi && (key0[h] >= lo || key0[h] + FRB_PAGE <= p.keep_first));
+#pragma unroll 1
+            for (int h = 0; h < pages; ++h) {
+                const int key0 = run_at(AP_STEP_PAGES * j + h, kept, first_page) * FRB_PAGE;
                 uint32_t raw[FRB_PAGE / 16][16];
 #pragma unroll
                 for (int c = 0; c < FRB_PAGE / 16; ++c) tmem_ld16(mine + 64 * h + 16 * c, raw[c]);
                 tmem_wait_ld();
-                if (open[h]) {
+                if (open_page(key0)) {
                     float top[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
                     for (int c = 0; c < FRB_PAGE / 16; ++c)
@@ -196,7 +196,7 @@ attention_pair_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                     for (int c = 0; c < FRB_PAGE / 16; ++c)
 #pragma unroll
                         for (int i = 0; i < 16; ++i)
-                            if (key_visible(key0[h] + 16 * c + i, lo, hi, p.keep_first)) step_max = fmaxf(step_max, __uint_as_float(raw[c][i]));
+                            if (key_visible(key0 + 16 * c + i, lo, hi, p.keep_first)) step_max = fmaxf(step_max, __uint_as_float(raw[c][i]));
                 }
             }
             if (step_max > -INFINITY) step_max = CAPPED ? capped_score2(step_max, p.cap_scale, p.cap2) : step_max * scale2;  // positive scale
@@ -217,20 +217,20 @@ attention_pair_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             l_sum *= corr;
             const float m_sub = m_used == -INFINITY ? 0.f : m_used;
             const uint64_t scale_pair = pair_of(scale2, scale2), shift_pair = pair_of(-m_sub, -m_sub);
-#pragma unroll
-            for (int h = 0; h < AP_STEP_PAGES; ++h) {
-                if (h >= pages) break;
+#pragma unroll 1
+            for (int h = 0; h < pages; ++h) {
+                const int key0 = run_at(AP_STEP_PAGES * j + h, kept, first_page) * FRB_PAGE;
                 uint32_t raw[FRB_PAGE / 16][16];
 #pragma unroll
                 for (int c = 0; c < FRB_PAGE / 16; ++c) tmem_ld16(mine + 64 * h + 16 * c, raw[c]);
                 tmem_wait_ld();
-                if (CAPPED) cap_scores(raw, p.cap_scale);
-                if (!open[h]) {
+                if (CAPPED) cap_scores(raw, p.cap_scale, p.cap2);
+                if (!open_page(key0)) {
 #pragma unroll
                     for (int c = 0; c < FRB_PAGE / 16; ++c)
 #pragma unroll
                         for (int i = 0; i < 16; ++i)
-                            if (!key_visible(key0[h] + 16 * c + i, lo, hi, p.keep_first)) raw[c][i] = 0xff800000u;      // minus infinity
+                            if (!key_visible(key0 + 16 * c + i, lo, hi, p.keep_first)) raw[c][i] = 0xff800000u;      // minus infinity
                 }
                 uint64_t sums[4] = {0ull, 0ull, 0ull, 0ull};
                 uint32_t packed[FRB_PAGE / 32][16];

@@ -212,9 +212,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
             for (int c = 0; c < FRB_PAGE / 16; ++c) tmem_ld16(mine + 16 * c, raw[c]);
             tmem_wait_ld();
-            // CAPPED: every score becomes tanh(score * scale / cap) first; what follows then sees a scale of cap * log2(e)
-            const float scale2 = CAPPED ? p.cap2 : p.scale2;
-            if (CAPPED) cap_scores(raw, p.cap_scale);
+            // CAPPED: every score becomes cap * tanh(score * scale / cap) * log2(e) first; what follows then sees a scale of one
+            const float scale2 = CAPPED ? 1.f : p.scale2;
+            if (CAPPED) cap_scores(raw, p.cap_scale, p.cap2);
             // Most pages lie wholly before the tile's first query (and inside the window): no key of theirs is
             // masked for any row of this warp, and the per-key comparisons are left out.
             const bool open_page = __all_sync(0xffffffffu, valid && key0 + FRB_PAGE - 1 <= hi && (key0 >= lo || key0 + FRB_PAGE <= p.keep_first));

@@ -50,14 +50,46 @@ __device__ __forceinline__ uint64_t mul_pairs(uint64_t a, uint64_t b) {
     return d;
 }
 
-// tanh(x) of a page's scores x = raw * cap_scale, in place.  Where no score of the warp's rows passes 0.4 of the cap: the
-// Taylor series x (1 - x^2/3 + 2 x^4/15 - 17 x^6/315 + 62 x^8/2835 - 1382 x^10/155925), whose next term is below 1e-7 of x
-// there, two scores at a time on the multiply-add pipe; else 1 - 2 / (exp(2x) + 1) with the hardware's exponential and
-// reciprocal (two trips to the special-function unit a score, beside the softmax's own).
-#define AT_SERIES_REACH 0.4f
+// Capped scores of a page, in place: cap2 * tanh(x) with x = raw * cap_scale (cap2 = cap * log2(e): the result is in units of
+// log2).  Where no score of the warp's rows passes a fifth of the cap, or two fifths, the Taylor series of tanh serves,
+//     x (1 - x^2/3 + 2 x^4/15 - 17 x^6/315 [+ 62 x^8/2835 - 1382 x^10/155925]),
+// its next term below 1e-7 of x there, as a polynomial in raw^2 with the scales in its coefficients, two scores at a time on the
+// multiply-add pipe; else 1 - 2 / (exp(2x) + 1) with the hardware's exponential and reciprocal (two trips to the special-function
+// unit a score, beside the softmax's own).
+template <int TERMS, int N>
+__device__ __forceinline__ void cap_by_series(uint32_t (&raw)[N][16], float cap_scale, float cap2) {
+    constexpr float series[6] = {1.0f, -1.0f / 3.0f, 2.0f / 15.0f, -17.0f / 315.0f, 62.0f / 2835.0f, -1382.0f / 155925.0f};
+    uint64_t k[TERMS];
+    float scale = cap_scale * cap2;
+#pragma unroll
+    for (int n = 0; n < TERMS; ++n) { k[n] = pair_of(series[n] * scale, series[n] * scale); scale *= cap_scale * cap_scale; }
+#pragma unroll
+    for (int c = 0; c < N; ++c) {
+        // eight pairs a stage: a pair's own chain of dependent operations would wait for itself
+        uint64_t x[8], x2[8], f[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            x[i] = pair_of(__uint_as_float(raw[c][2 * i]), __uint_as_float(raw[c][2 * i + 1]));
+            x2[i] = mul_pairs(x[i], x[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = fma_pairs(x2[i], k[TERMS - 1], k[TERMS - 2]);
+#pragma unroll
+        for (int n = TERMS - 3; n >= 0; --n)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) f[i] = fma_pairs(x2[i], f[i], k[n]);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            float lo, hi;
+            halves_of(mul_pairs(x[i], f[i]), lo, hi);
+            raw[c][2 * i] = __float_as_uint(lo);
+            raw[c][2 * i + 1] = __float_as_uint(hi);
+        }
+    }
+}
 
 template <int N>
-__device__ __forceinline__ void cap_scores(uint32_t (&raw)[N][16], float cap_scale) {
+__device__ __forceinline__ void cap_scores(uint32_t (&raw)[N][16], float cap_scale, float cap2) {
     float top[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
     for (int c = 0; c < N; ++c)
@@ -65,34 +97,15 @@ __device__ __forceinline__ void cap_scores(uint32_t (&raw)[N][16], float cap_sca
         for (int i = 0; i < 16; i += 2)
             top[(i >> 1) & 3] = max3(top[(i >> 1) & 3], fabsf(__uint_as_float(raw[c][i])), fabsf(__uint_as_float(raw[c][i + 1])));
     const float most = fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3])) * cap_scale;
-    if (__all_sync(0xffffffffu, most <= AT_SERIES_REACH)) {
-        const uint64_t scale = pair_of(cap_scale, cap_scale), one = pair_of(1.f, 1.f);
-        const float k1 = -1.0f / 3.0f, k2 = 2.0f / 15.0f, k3 = -17.0f / 315.0f, k4 = 62.0f / 2835.0f, k5 = -1382.0f / 155925.0f;
-        const uint64_t c1 = pair_of(k1, k1), c2 = pair_of(k2, k2), c3 = pair_of(k3, k3), c4 = pair_of(k4, k4), c5 = pair_of(k5, k5);
-#pragma unroll
-        for (int c = 0; c < N; ++c)
-#pragma unroll
-            for (int i = 0; i < 16; i += 2) {
-                const uint64_t x = mul_pairs(pair_of(__uint_as_float(raw[c][i]), __uint_as_float(raw[c][i + 1])), scale);
-                const uint64_t x2 = mul_pairs(x, x);
-                uint64_t f = fma_pairs(x2, c5, c4);
-                f = fma_pairs(x2, f, c3);
-                f = fma_pairs(x2, f, c2);
-                f = fma_pairs(x2, f, c1);
-                f = fma_pairs(x2, f, one);
-                float lo, hi;
-                halves_of(mul_pairs(x, f), lo, hi);
-                raw[c][i] = __float_as_uint(lo);
-                raw[c][i + 1] = __float_as_uint(hi);
-            }
+    if (__all_sync(0xffffffffu, most <= 0.2f)) {
+        cap_by_series<4>(raw, cap_scale, cap2);
+    } else if (__all_sync(0xffffffffu, most <= 0.4f)) {
+        cap_by_series<6>(raw, cap_scale, cap2);
     } else {
 #pragma unroll
         for (int c = 0; c < N; ++c)
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-                const float e = exp2f(fminf(__uint_as_float(raw[c][i]) * cap_scale, 40.f) * 2.8853900817779268f);
-                raw[c][i] = __float_as_uint(1.0f - __fdividef(2.0f, e + 1.0f));
-            }
+            for (int i = 0; i < 16; ++i) raw[c][i] = __float_as_uint(capped_score2(__uint_as_float(raw[c][i]), cap_scale, cap2));
     }
 }
 

@@ -579,7 +579,45 @@ def duzinex(kind: str, launches: int) -> dict:
     return {"case": kind, "tokens": tokens, "ms": round(ms, 4), "gbs": round((moved + state_bytes) / ms / 1e6, 1)}
 
 
+def attention_of_two_maps(kind: str, launches: int) -> dict:
+    """Prompt attention with two maps of 64 entries per head, 16 heads over 4 value heads of 128, scores capped at 30: four prompts of
+    2,048 tokens with a window of 1,024 beside four first tokens (``long``: one prompt of 16,384 without a window).  ``two``: a map
+    a block in float32 and the difference in a kernel of its own; ``plain``: no cap."""
+    heads, v_heads, dim, vdim = 16, 4, 64, 128
+    long = "long" in kind
+    lengths, window = ([16384], None) if long else ([2048] * 4, 1024)
+    tokens, pages = sum(lengths), sum(n // 64 for n in lengths)
+    q = torch.randn(tokens, 2 * heads * dim, device=DEV).to(torch.bfloat16)
+    k = torch.randn(pages, 2 * v_heads, 64, dim, device=DEV).to(torch.bfloat16)
+    v = torch.randn(pages, v_heads, vdim, 64, device=DEV).to(torch.bfloat16)
+    table = torch.arange(pages, dtype=torch.int32, device=DEV).view(len(lengths), -1).contiguous()
+    tiles = [(b, i) for b, n in enumerate(lengths) for i in range(0, n, 128)]
+    tile_seq, tile_q0 = (torch.tensor([t[i] for t in tiles], dtype=torch.int32, device=DEV) for i in range(2))
+    t = _Tables(lengths)
+    q_len = torch.tensor(lengths, dtype=torch.int32, device=DEV)
+    out = torch.empty(tokens, heads * vdim, dtype=torch.bfloat16, device=DEV)
+    maps = torch.empty(tokens, 2 * heads * vdim, device=DEV)
+    lam = torch.full((1,), 0.5, device=DEV)
+    cap = None if "plain" in kind else 30.0
+    tables = (table, tile_seq, tile_q0, t.seq_slot, t.seq_start, q_len, t.cu_q_len)
+
+    def launch():
+        if "two" in kind:
+            ops.attention_prefill_tc(q, k, v, *tables, maps, num_heads=2 * heads, num_kv_heads=2 * v_heads, head_dim=dim, v_dim=vdim,
+                                     scale=dim ** -0.5, window=window, keep_first=4, softcap=cap, maps=2)
+            ops.map_difference(maps, out, heads=heads, kv_heads=v_heads, v_dim=vdim, lam=lam, eps=1e-6, factor=0.5)
+        else:
+            ops.attention_pair_tc(q, k, v, *tables, out, heads=heads, v_heads=v_heads, head_dim=dim, v_dim=vdim, scale=dim ** -0.5,
+                                  window=window, keep_first=4, softcap=cap, lam=lam, eps=1e-6, factor=0.5)
+    ms = _time(launch, launches)
+    ops.tc_status_check(DEV)
+    seen = sum(min(i + 1, window or i + 1) for n in lengths for i in range(n))
+    return {"case": f"maps_{kind}", "tokens": tokens, "ms": round(ms, 4), "tflops": round(2.0 * 2 * heads * seen * (dim + vdim) / ms / 1e9, 1)}
+
+
 CASES = {
+    **{f"maps_{kind}": (lambda n, kind=kind: attention_of_two_maps(kind, n))
+       for kind in ("prefill", "prefill_plain", "prefill_two", "prefill_two_plain", "long", "long_plain", "long_two", "long_two_plain")},
     **{f"duzinex_{kind}": (lambda n, kind=kind: duzinex(kind, n))
        for kind in ("retention_prefill", "retention_decode", "gru_prefill", "gru_decode", "shift_prefill", "shift_decode",
                     "powers_prefill", "powers_decode")},
