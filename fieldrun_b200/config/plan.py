@@ -42,6 +42,8 @@ class LayerSpec:
     feed_forward_out_norm: Optional[PartSpec] = None
     # a part between the mixer's norm and the mixer (category ``mixer_input``), which may keep a state of its own
     mixer_input: Optional[PartSpec] = None
+    # how the sublayers read and write a stream that is kept as several copies (category ``stream_connection``)
+    connections: Optional[PartSpec] = None
 
 
 @dataclass(frozen=True)
@@ -71,8 +73,15 @@ class ModelPlan:
     head: PartSpec
     eos_token_id: tuple[int, ...] = ()
     connectors: tuple[PartSpec, ...] = ()
+    # copies of the residual stream that the layers' connections work on, all equal to the embedding's rows at the start
+    # and added up in front of the final norm; 0: one plain stream
+    streams: int = 0
 
     def check(self) -> None:
+        if self.streams < 0 or any((layer.connections is not None) != (self.streams > 0) for layer in self.layers):
+            raise ValueError(f"a plan with {self.streams} copies of the stream: every layer has connections to them, or, with 0, none")
+        if self.streams and (self.connectors or any(layer.addition is not None for layer in self.layers)):
+            raise ValueError("connectors and additions work on a single stream, not on copies of it")
         written: set[int] = set()
         for step, run in enumerate(self.run_order):
             if run.connector is not None and not 0 <= run.connector[0] < len(self.connectors):

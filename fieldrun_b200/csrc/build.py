@@ -39,6 +39,7 @@ GROUPS: dict[str, tuple[str, ...]] = {
     "scans": ("scans.cu",),
     "delta": ("delta_rule.cu",),
     "retention": ("retention.cu",),
+    "copies": ("stream_copies.cu",),
     "latent": ("latent_attention.cu", "latent_attention_tc.cu"),
     "extras": ("attention_decode_noalloc.cu", "wait_probe.cu"),
 }

@@ -217,8 +217,8 @@ FRB_API int frb_rmsnorm(float* x, const float* delta, const float* expert_y, con
 // ----------------------------------------------------------------------------- Q/K norm + rotary + cache write
 
 struct QkvParams {
-    const void* qkv;          // [T, (nh + nkv) * hd + nvh * vd], InT
-    const float* bias;        // [(nh + nkv) * hd + nvh * vd] added to the row before anything else, or null
+    const void* qkv;          // [T, (nh + nkv) * hd + nvh * vd], InT; without the value columns where the values are the keys
+    const float* bias;        // as wide as a row, added to it before anything else, or null
     const void* q_weight;     // [nh*hd] or null: no norm
     const void* k_weight;     // [nkv*hd] or null
     const float* cos_table;   // [positions, rotary_dim/2]
@@ -238,6 +238,9 @@ struct QkvParams {
     int v_dim;                // size of a value head (the keys' head_dim unless the design says otherwise)
     int num_v_heads;          // value heads (the number of key heads unless several of those share one)
     unsigned v_dim_inverse;
+    int v_from;               // the row's column where the values begin: behind the keys, or the keys' own (values that are
+                              // the keys before their rotation)
+    int row_width;            // columns of a row
     float q_temp_coef;        // the query is multiplied by 1 + coef * ln(floor((pos + 1) / every) + 1); 0: no such factor
     int q_temp_every;
 };
@@ -261,7 +264,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_kernel(QkvParams p) {
     const int hd = p.head_dim;
     const int q_width = p.num_heads * hd, k_width = p.num_kv_heads * hd;
     const int vd = p.v_dim, v_width = p.num_v_heads * vd;
-    const int qk_width = q_width + k_width, all_width = qk_width + v_width;
+    const int qk_width = q_width + k_width, all_width = p.row_width;
     const int half = p.rotary_dim / 2;
     float* s_cos = raw + all_width;
     float* s_sin = s_cos + half;
@@ -343,7 +346,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_kernel(QkvParams p) {
         }
     }
     if (page >= 0) {
-        const float* vrow = raw + qk_width;
+        const float* vrow = raw + p.v_from;
         for (int i = threadIdx.x; i < v_width; i += NORM_BLOCK) {
             const int head = i / vd, dim = i - head * vd;
             const size_t at = (((size_t)page * p.num_v_heads + head) * vd + dim) * FRB_PAGE + in_page;
@@ -365,7 +368,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_vec_kernel(QkvParams p
     const int hd = p.head_dim;
     const int q_width = p.num_heads * hd, k_width = p.num_kv_heads * hd;
     const int vd = p.v_dim, v_width = p.num_v_heads * vd;
-    const int qk_width = q_width + k_width, all_width = qk_width + v_width;
+    const int qk_width = q_width + k_width, all_width = p.row_width;
     int pos_early = 0, slot_early = 0, page_early = -1;
     // the blocks that transpose values come first in the grid: they run longest, and at the grid's end they ran alone
     const int token_block = (int)blockIdx.x - p.v_tiles;
@@ -399,8 +402,8 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_vec_kernel(QkvParams p
         // a warp reads a token's dimensions, then writes a dimension's tokens: no division per element
         const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
         for (int j = warp; j < count; j += NORM_BLOCK / 32) {
-            const InT* row = (const InT*)p.qkv + (size_t)(t0 + j) * all_width + qk_width + h * vd;
-            const float* brow = p.bias ? p.bias + qk_width + h * vd : nullptr;
+            const InT* row = (const InT*)p.qkv + (size_t)(t0 + j) * all_width + p.v_from + h * vd;
+            const float* brow = p.bias ? p.bias + p.v_from + h * vd : nullptr;
             for (int d = lane; d < vd; d += 32)
                 tile[d * (QKV_V_TOKENS + 2) + j] = from_f32<OutT>(to_f32<InT>(row[d]) + (brow ? brow[d] : 0.f));
         }
@@ -499,7 +502,7 @@ __global__ void __launch_bounds__(NORM_BLOCK) qkv_prepare_vec_kernel(QkvParams p
         }
     }
     if (page >= 0 && !p.v_tiles) {
-        const float* vrow = raw + qk_width;
+        const float* vrow = raw + p.v_from;
         for (int i = threadIdx.x; i < v_width; i += NORM_BLOCK) {
             const int head = (int)__umulhi((unsigned)i, p.v_dim_inverse), dim = i - head * vd;
             const size_t at = (((size_t)page * p.num_v_heads + head) * vd + dim) * FRB_PAGE + in_page;
@@ -514,12 +517,14 @@ FRB_API int frb_qkv_prepare(const void* qkv, int in_dtype, const void* q_weight,
                             void* q_out, void* k_pages, void* v_pages, int out_dtype, int num_tokens, int num_heads,
                             int num_kv_heads, int head_dim, int rotary_dim, int interleaved, int write_cache,
                             int per_head, int tables_final, const float* bias, int v_dim, float q_temp_coef,
-                            int q_temp_every, int num_v_heads, cudaStream_t stream) {
+                            int q_temp_every, int num_v_heads, int values_from_keys, cudaStream_t stream) {
     if (num_tokens == 0) return 0;
     if (v_dim <= 0) v_dim = head_dim;
     if (num_v_heads < 0) num_v_heads = num_kv_heads;
     FRB_CHECK_ARG(num_v_heads == num_kv_heads || (num_v_heads > 0 && num_kv_heads % num_v_heads == 0),
                   "qkv_prepare: %d key heads over %d value heads", num_kv_heads, num_v_heads);
+    FRB_CHECK_ARG(!values_from_keys || (!k_weight && v_dim == head_dim && num_v_heads == num_kv_heads),
+                  "qkv_prepare: values that are the keys as projected go without a norm of the keys and have the keys' heads and size");
     FRB_CHECK_ARG(q_temp_coef == 0.f || q_temp_every >= 1, "qkv_prepare: a query temperature every %d positions", q_temp_every);
     FRB_CHECK_ARG(rotary_dim % 2 == 0 && rotary_dim <= head_dim, "qkv_prepare: rotary_dim %d must be even and <= head_dim %d",
                   rotary_dim, head_dim);
@@ -535,8 +540,10 @@ FRB_API int frb_qkv_prepare(const void* qkv, int in_dtype, const void* q_weight,
     p.head_dim_inverse = (unsigned)((0x100000000ull + (unsigned)head_dim - 1) / (unsigned)head_dim);
     p.bias = bias; p.v_dim = v_dim; p.num_v_heads = num_v_heads; p.q_temp_coef = q_temp_coef; p.q_temp_every = q_temp_every > 0 ? q_temp_every : 1;
     p.v_dim_inverse = (unsigned)((0x100000000ull + (unsigned)v_dim - 1) / (unsigned)v_dim);
-    const long long all_width = (long long)(num_heads + num_kv_heads) * head_dim + (long long)num_v_heads * v_dim;
+    const long long all_width = (long long)(num_heads + num_kv_heads) * head_dim + (values_from_keys ? 0ll : (long long)num_v_heads * v_dim);
     FRB_CHECK_ARG(all_width < (1 << 24), "qkv_prepare: %d heads of %d", num_heads, head_dim);
+    p.row_width = (int)all_width;
+    p.v_from = (num_heads + (values_from_keys ? 0 : num_kv_heads)) * head_dim;
     // per-head statistics: the squares of the q and k rows and one factor per head beside the rows
     const size_t smem = ((size_t)all_width + rotary_dim +
                          (p.per_head ? (size_t)(num_heads + num_kv_heads) * (head_dim + 1) : 0)) * sizeof(float);
@@ -662,16 +669,19 @@ FRB_API int frb_unary_unit(const float* in, void* out, int out_dtype, long long 
     FRB_RETURN_LAUNCH("unary_unit");
 }
 
-// x[i] = cap * tanh(x[i] / cap), in place on float32 logits.
-__global__ void softcap_kernel(float* __restrict__ x, float cap, size_t total) {
+// x[i] = cap * tanh(scale * x[i] / cap), in place on float32 logits; without a cap (0) only scale * x[i].
+__global__ void softcap_kernel(float* __restrict__ x, float cap, float scale, size_t total) {
     after_previous_kernel();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < total) x[i] = cap * tanhf(x[i] / cap);
+    if (i < total) {
+        const float z = scale * x[i];
+        x[i] = cap > 0.f ? cap * tanhf(z / cap) : z;
+    }
 }
 
-FRB_API int frb_softcap(float* x, long long total, float cap, cudaStream_t stream) {
+FRB_API int frb_softcap(float* x, long long total, float cap, float scale, cudaStream_t stream) {
     if (total == 0) return 0;
-    FRB_CHECK_ARG(cap > 0.f, "softcap: a cap of %f", (double)cap);
-    launch_dependent(softcap_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, x, cap, (size_t)total);
+    FRB_CHECK_ARG(cap >= 0.f, "softcap: a cap of %f", (double)cap);
+    launch_dependent(softcap_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, x, cap, scale, (size_t)total);
     FRB_RETURN_LAUNCH("softcap");
 }

@@ -22,13 +22,13 @@ _P, _I, _F, _L = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlon
 _SIGNATURES = {
     "frb_embed_rows": "ppipiiifpi",
     "frb_rmsnorm": "pppppippifiipipi",
-    "frb_qkv_prepare": "pippifppipppipppiiiiiiiiiipifii",
+    "frb_qkv_prepare": "pippifppipppipppiiiiiiiiiipifiii",
     "frb_wait_probe": "lpp",
     "frb_add_rows": "ppl",
     "frb_attention_generic": "pppipipppiiiifiipippif" "iii",
     "frb_layernorm": "ppppfppiii",
     "frb_unary_unit": "ppili",
-    "frb_softcap": "plf",
+    "frb_softcap": "plff",
     "frb_dyt_norm": "ppppppippppppppppiiii",
     "frb_rms_blend": "pppppiiff",
     "frb_concat_rows": "ppppiiii",
@@ -65,6 +65,7 @@ _SIGNATURES = {
     "frb_attention_prefill_tc": "pippipippipppppiiifippipf" "iiii",
     "frb_attention_pair_tc": "pippi" "pippi" "ppppp" "iiiifiif" "pffp",
     "frb_dyt_rows": "ppppp" "ppp" "pp" "iii" "p" "pppp" "pll",
+    "frb_stream_copies": "pip" "pp" "ppppp" "ip" "ppp" "ppp" "pip" "iii",
     "frb_map_difference": "pppi" "iiiiff",
     "frb_poly_norm": "pppiiif",
     "frb_min_gru": "piiii" "pp" "ppp" "pll" "pi" "iii",
@@ -108,6 +109,7 @@ _ENTRY_GROUPS = {
               "frb_min_gru"),
     "delta": ("frb_gated_delta_rule",),
     "retention": ("frb_retention",),
+    "copies": ("frb_stream_copies",),
     "extras": ("frb_wait_probe",),
 }
 _GROUP_OF = {entry: group for group, entries in _ENTRY_GROUPS.items() for entry in entries}
@@ -307,10 +309,10 @@ def unary_unit(rows_in: torch.Tensor, out: torch.Tensor, activation: str) -> Non
     _call("frb_unary_unit", _ptr(rows_in), _ptr(out), _code(out.dtype), rows_in.numel(), ACTIVATIONS[activation])
 
 
-def softcap(logits: torch.Tensor, cap: float) -> None:
-    """logits <- cap * tanh(logits / cap), in place."""
+def softcap(logits: torch.Tensor, cap: Optional[float], scale: float = 1.0) -> None:
+    """logits <- cap * tanh(scale * logits / cap), in place; without a cap only scale * logits."""
     _want(logits, torch.float32, "logits")
-    _call("frb_softcap", _ptr(logits), logits.numel(), float(cap))
+    _call("frb_softcap", _ptr(logits), logits.numel(), float(cap or 0.0), float(scale))
 
 
 def gla_scan(proj: torch.Tensor, offsets: tuple[int, int, int, int, int], a2: torch.Tensor, a2_bias: torch.Tensor,
@@ -436,6 +438,49 @@ def dyt_rows(x: torch.Tensor, norm: tuple[torch.Tensor, torch.Tensor, torch.Tens
     _call("frb_dyt_rows", _ptr(x), _ptr(deltas[0]) if deltas else None, _ptr(deltas[1]) if len(deltas) > 1 else None, _ptr(vector),
           _ptr(rows), _ptr(norm[0]), _ptr(norm[1]), _ptr(norm[2]), _ptr(stream), _ptr(out), _code(out.dtype), num_rows, x.shape[-1],
           *_shift_args(shift))
+
+
+STREAM_COPIES = 64             # most copies of the stream (COPIES_MAX_STREAMS)
+COPIES_MAX_SUMMED_ROWS = 64    # most weighted rows per token that the kernel sums itself (COPIES_MAX_TOP_K)
+
+
+def stream_copies(x: torch.Tensor, streams: int, *, first: Optional[tuple[torch.Tensor, torch.Tensor]] = None, second: tuple = (),
+                  experts=None, second_out: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                  gather: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, norm=None,
+                  store: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, out32: Optional[torch.Tensor] = None) -> None:
+    """The copies of a stream between two sublayers: v_t = sum_s mix[s, t] x_s + oa[t] ya + ob[t] yb, u = sum_t gather[t] v_t.
+    ``x`` [T, streams, width], or [T, width] for copies that are all equal; ``first`` = (ya, oa); yb is the sum of ``second``
+    (up to two float32 tensors) and of ``experts`` = (y, weights, row_of_assign), ``second_out`` = ob; without ``mix`` the
+    copies stay, without ``gather`` they are added up.  ``store`` gets the v (x itself, or another buffer).  ``out`` and
+    ``out32`` get u, or with ``norm`` = (w, b, alpha) its dynamic tanh; ``rows`` picks rows of x and the updates."""
+    second = tuple(d for d in second if d is not None)
+    for t in (x, mix, gather, store, out32, second_out, *(first or ()), *second, *(norm or ())):
+        if t is not None:
+            _want(t, torch.float32, "the stream's copies, their updates and constants")
+    count, width = x.shape[0], x.shape[-1]
+    if x.dim() not in (2, 3) or (x.dim() == 3 and x.shape[1] != streams):
+        raise KernelError(f"a stream of {streams} copies of shape {tuple(x.shape)}")
+    if len(second) > 2 or any(tuple(t.shape) != (count, width) for t in ((first[0],) if first else ()) + second):
+        raise KernelError("stream_copies adds tensors of one row of the stream's width a token, two to the second update")
+    if store is not None and tuple(store.shape) != (count, streams, width):
+        raise KernelError(f"the copies go into a buffer of shape {tuple(store.shape)}")
+    if (mix is not None and tuple(mix.shape) != (streams, streams)) or any(
+            t is not None and t.numel() != streams for t in (gather, second_out, first[1] if first else None)):
+        raise KernelError(f"constants that are not made for {streams} copies")
+    if rows is not None:
+        _want(rows, torch.int32, "row indices")
+    y = ew = rowmap = None
+    if experts is not None:
+        y, ew, rowmap = experts
+        _want(y, torch.float32, "expert outputs")
+        _want(ew, torch.float32, "expert weights")
+        _want(rowmap, torch.int32, "rows of the assignments")
+    w, b, alpha = norm if norm is not None else (None, None, None)
+    _call("frb_stream_copies", _ptr(x), int(x.dim() == 2), _ptr(store), _ptr(first[0]) if first else None,
+          _ptr(first[1]) if first else None, _ptr(second[0]) if second else None, _ptr(second[1]) if len(second) > 1 else None, _ptr(y),
+          _ptr(ew), _ptr(rowmap), ew.shape[-1] if ew is not None else 0, _ptr(second_out), _ptr(mix), _ptr(gather), _ptr(rows), _ptr(w),
+          _ptr(b), _ptr(alpha), _ptr(out), _code(out.dtype) if out is not None else 0, _ptr(out32),
+          rows.numel() if rows is not None else count, width, streams)
 
 
 def token_shift(h: torch.Tensor, out: torch.Tensor, *, shift) -> None:
@@ -691,7 +736,7 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
                 num_kv_heads: int, head_dim: int, rotary_dim: int, interleaved: bool, write_cache: bool,
                 per_head: bool = False, tables_final: bool = False, bias: Optional[torch.Tensor] = None,
                 v_dim: Optional[int] = None, q_temp: Optional[tuple[float, int]] = None,
-                num_v_heads: Optional[int] = None) -> None:
+                num_v_heads: Optional[int] = None, values_from_keys: bool = False) -> None:
     """Q/K RMSNorm (when weights are given: over the whole row with weights [heads * head_dim], or with
     ``per_head`` over each head with weights [head_dim]), rotary from the tables, Q out, K/V into their pages.
     ``tables_final``: positions, slots and the page table were complete before the kernel before this one in
@@ -699,7 +744,8 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
     them, and the angles, while that kernel still runs.  ``bias`` (float32, as wide as a row of ``qkv``) is added
     first; ``v_dim`` is the size of a value head if it is not ``head_dim``, ``num_v_heads`` their number if it is not
     ``num_kv_heads``; ``q_temp`` = (coef, every) multiplies the
-    query at position p by 1 + coef * ln(floor((p + 1) / every) + 1).  A row without keys and values (a layer that
+    query at position p by 1 + coef * ln(floor((p + 1) / every) + 1).  ``values_from_keys``: a row has no value columns, the
+    values are the keys as projected, before rotation (and without a norm of the keys).  A row without keys and values (a layer that
     reads another layer's cache line) is ``num_kv_heads = 0`` with ``write_cache`` false."""
     if (q_weight is None) != (k_weight is None) and num_kv_heads > 0:
         raise KernelError("q and k norm weights come together or not at all")
@@ -722,7 +768,7 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
           _ptr(q_out), _ptr(k_pages), _ptr(v_pages), _code(out_dtype), qkv.shape[0], num_heads, num_kv_heads, head_dim,
           rotary_dim, int(interleaved), int(write_cache), int(per_head), int(tables_final), _ptr(bias),
           int(v_dim or head_dim), float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 1,
-          -1 if num_v_heads is None else int(num_v_heads))
+          -1 if num_v_heads is None else int(num_v_heads), int(values_from_keys))
 
 
 def attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, page_table: torch.Tensor,

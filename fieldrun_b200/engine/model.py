@@ -53,6 +53,8 @@ class DecoderModel:
         for block, layer in zip(self.blocks, plan.layers):
             if layer.mixer_input is not None:
                 block.set_mixer_input(build_part("mixer_input", layer.mixer_input, self.dtype))
+            if layer.connections is not None:
+                block.set_connections(build_part("stream_connection", layer.connections, self.dtype))
         self.additions = [build_part("addition", layer.addition, self.dtype) if layer.addition is not None else None
                           for layer in plan.layers]
         self.connectors = [build_part("connector", spec, self.dtype) for spec in plan.connectors]
@@ -182,5 +184,8 @@ class DecoderModel:
                 x, pending = self.additions[run.layer].forward(ctx, x, pending)
         if logit_rows is None or logit_rows.numel() == 0:
             return None
+        if self.plan.streams:                           # the copies of the stream end as their sum
+            _, act, _ = self.final_norm.forward_copies(ctx, x, pending, self.plan.streams, rows=logit_rows)
+            return self.head.forward(ctx, act)
         act, _ = self.final_norm.forward(ctx, x, delta=pending, rows=logit_rows, write_back=False)
         return self.head.forward(ctx, act)

@@ -1,2 +1,2 @@
 """Built-in architectures; importing this package registers them."""
-from . import bakasun, bamasun, depelix, duzinex, fotanex, minimax_m2  # noqa: F401
+from . import bakasun, bamasun, depelix, duzinex, fotanex, kifunex, minimax_m2  # noqa: F401

@@ -24,7 +24,8 @@ sigmoid(W_g x)_h, one row of W_g per head, before the output projection), ``sink
 every head instead of a learned tensor: 0.0 adds one to the softmax's denominator), ``softcap`` (the scaled score s
 of every key becomes softcap * tanh(s / softcap) before the softmax), ``keep_first`` (beside a window, the sequence's first
 tokens stay visible to every query, at their true positions; the cache keeps their pages), ``output_bias`` (the output
-projection has a bias, left to the norm that takes the update), ``differential`` ``{"diff", "eps"}``: every head has two maps,
+projection has a bias, left to the norm that takes the update), ``values_from_keys`` (there is no value projection: the values
+are the keys as projected, before the rotation), ``differential`` ``{"diff", "eps"}``: every head has two maps,
 each an attention of its own with queries and keys of ``head_dim`` over the same values, and gives
 
     o = a1 - lambda a2,   out = o / sqrt(mean(o^2) + eps) * (1 - diff)   (over the head's value entries),
@@ -65,6 +66,7 @@ class GQAAttention(Mixer):
         self.value_dim = int(a.get("value_dim") or self.head_dim)
         self.has_bias = bool(a.get("bias", False))
         self.shares_kv = bool(a.get("shares_kv", False))
+        self.values_from_keys = bool(a.get("values_from_keys", False))
         temperature = a.get("query_temperature")
         self.q_temp = (float(temperature["coef"]), int(temperature["every"])) if temperature else None
         if self.q_temp is not None and self.q_temp[1] < 1:
@@ -108,6 +110,9 @@ class GQAAttention(Mixer):
         if differential and (self.qk_norm != "none" or self.shares_kv or self.has_head_gate or self.has_sink
                              or self.sink_value is not None or self.slope_values is not None):
             raise ValueError("differential attention is built without q/k norms, shared keys, head gates, sinks and distance slopes")
+        if self.values_from_keys and (self.value_dim != self.head_dim or self.qk_norm != "none" or differential):
+            raise ValueError("values that are the keys as projected have the keys' size and go without a norm of the keys and without "
+                             "a second map")
         if self.num_heads % self.num_kv_heads:
             raise ValueError(f"{self.num_heads} heads are not a multiple of {self.num_kv_heads} kv heads")
         if not 1 <= self.head_dim <= 256:
@@ -139,12 +144,14 @@ class GQAAttention(Mixer):
         needs = {
             "q_proj": TensorNeed(self.name_of("q_proj"), (self.q_width, self.hidden_size), MATRIX, "normal"),
             "k_proj": TensorNeed(self.name_of("k_proj"), (self.kv_width, self.hidden_size), MATRIX, "normal"),
-            "v_proj": TensorNeed(self.name_of("v_proj"), (self.v_width, self.hidden_size), MATRIX, "normal"),
             "o_proj": TensorNeed(self.name_of("o_proj"), (self.hidden_size, self.out_width), MATRIX, "normal"),
         }
+        if not self.values_from_keys:
+            needs["v_proj"] = TensorNeed(self.name_of("v_proj"), (self.v_width, self.hidden_size), MATRIX, "normal")
         if self.has_bias:
             needs["q_bias"] = TensorNeed(self.name_of("q_bias"), (self.q_width,), VECTOR, "bias")
             needs["k_bias"] = TensorNeed(self.name_of("k_bias"), (self.kv_width,), VECTOR, "bias")
+        if self.has_bias and not self.values_from_keys:
             needs["v_bias"] = TensorNeed(self.name_of("v_bias"), (self.v_width,), VECTOR, "bias")
         if self.has_output_bias:
             needs["o_bias"] = TensorNeed(self.name_of("o_bias"), (self.hidden_size,), VECTOR, "bias")
@@ -171,11 +178,11 @@ class GQAAttention(Mixer):
 
     def load(self, source: TensorSource) -> None:
         needs = self._needs()
-        projections = ("q_proj",) if self.shares_kv else ("q_proj", "k_proj", "v_proj")
+        projections = tuple(n for n in ("q_proj", "k_proj", "v_proj") if n in needs)
         self.w_qkv = torch.cat([self._map_order(n, source.fetch(needs[n])) for n in projections], dim=0).contiguous()
         self.w_o = source.fetch(needs["o_proj"])
         if self.has_bias:
-            biases = ("q_bias",) if self.shares_kv else ("q_bias", "k_bias", "v_bias")
+            biases = tuple(n for n in ("q_bias", "k_bias", "v_bias") if n in needs)
             self.b_qkv = torch.cat([self._map_order(n, source.fetch(needs[n])) for n in biases], dim=0).contiguous()
         if self.has_output_bias:
             self.b_o = source.fetch(needs["o_bias"])
@@ -219,7 +226,7 @@ class GQAAttention(Mixer):
         tokens = act.shape[0]
         if self.shares_kv and writes_cache:
             raise ValueError("an attention layer without keys and values of its own was asked to write a cache line")
-        qkv = linear(act, self.w_qkv)                                        # float32 [T, q + k + v] (or [T, q])
+        qkv = linear(act, self.w_qkv)                                        # float32 [T, q + k + v] (or [T, q + k], [T, q])
         q = ctx.buffer("attention.q", (tokens, self.q_width), self.dtype)
         rotary_dim = self.position.rotary_dim if self.position is not None else 0
         ops.qkv_prepare(qkv, self.q_norm, self.k_norm, self.qk_norm_eps, self.cos, self.sin, ctx.tok_pos, ctx.tok_slot,
@@ -230,7 +237,8 @@ class GQAAttention(Mixer):
                         interleaved=bool(self.position.interleaved) if self.position is not None else False,
                         write_cache=writes_cache, per_head=self.qk_norm == "per_head",
                         tables_final=True,      # the step's tables were there before the projection above began
-                        bias=self.b_qkv, v_dim=self.value_dim, q_temp=self.q_temp)
+                        bias=self.b_qkv, v_dim=self.value_dim, q_temp=self.q_temp,
+                        values_from_keys=self.values_from_keys and not self.shares_kv)
         out = ctx.buffer("attention.out", (tokens, self.out_width), self.dtype)
         gate = linear(act, self.w_gate) if self.has_head_gate else None          # float32 [T, heads], before the sigmoid
         self.attend(ctx, q, line, out, gate)

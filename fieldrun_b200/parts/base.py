@@ -22,6 +22,8 @@ Interfaces
     the other place of a norm: x <- x + norm(update), for blocks whose sublayers read x itself.
 ``Norm.normed(ctx, update)`` -> norm(update) in float32
     a norm behind a sublayer whose block also has one in front (``NormedUpdate`` carries the pair to the next norm).
+``Norm.forward_copies(ctx, x, update, streams, gather=..., store=...)`` -> (x, rows, rows in float32)
+    the norm of a weighted sum of the copies of a stream that is kept several times (blocks with hyper-connections).
 ``Connector.forward(ctx, x, pending, first, index)`` -> the new stream [T, width] (float32)
     a part between two runs that rewrites the whole stream; ``first`` holds the embedding's rows.
     ``forward_deferred`` -> (stream, pending): for one that only adds and may leave the sum to the next norm.
@@ -177,6 +179,32 @@ class NormedUpdate(DeferredUpdate):
         return self.norm.normed(ctx, as_tensor(ctx, self.inner))
 
 
+class CopiesUpdate:
+    """What sublayers left for a stream that is kept as several copies: v_t = sum_s mix[s, t] x_s + first_out[t] * first +
+    second_out[t] * second.  ``first`` and ``second`` are float32 tensors [T, width] or any deferred form (or None); ``mix``
+    [S, S] and the weights [S] are float32 tensors on the device."""
+
+    def __init__(self, mix: torch.Tensor, first=None, first_out: Optional[torch.Tensor] = None, second=None,
+                 second_out: Optional[torch.Tensor] = None):
+        self.mix, self.first, self.first_out, self.second, self.second_out = mix, first, first_out, second, second_out
+
+    def kernel_args(self, ctx) -> dict:
+        """The update as ``ops.stream_copies`` takes it: its first part one tensor, its second one summed there if it can be."""
+        from ..csrc import ops
+        tensors, experts = (), None
+        second = self.second
+        if isinstance(second, WeightedRows) and second.top_k <= ops.COPIES_MAX_SUMMED_ROWS:
+            experts = (second.rows, second.weights, second.row_map)
+        elif (isinstance(second, UpdateSum) and second.vector is None and len(second.tensors) <= 2
+                and all(w.top_k <= ops.COPIES_MAX_SUMMED_ROWS for w in second.weighted)):
+            tensors = tuple(second.tensors)
+            experts = next(((w.rows, w.weights, w.row_map) for w in second.weighted), None)
+        elif second is not None:
+            tensors = (as_tensor(ctx, second),)
+        first = (as_tensor(ctx, self.first), self.first_out) if self.first is not None else None
+        return dict(mix=self.mix, first=first, second=tensors, experts=experts, second_out=self.second_out)
+
+
 def as_tensor(ctx, update):
     """The update as a float32 tensor, whatever form it came in (None stays None)."""
     return update.materialize(ctx) if isinstance(update, DeferredUpdate) else update
@@ -197,6 +225,27 @@ class Norm(Part):
     def normed(self, ctx, update: torch.Tensor) -> torch.Tensor:
         """norm(update) as a float32 tensor [T, width]: the norm of rows that are not the stream (a sublayer's output)."""
         raise NotImplementedError(f"norm {self.spec.kind!r} has no form that norms rows other than the stream")
+
+
+    def forward_copies(self, ctx, x: torch.Tensor, update: Optional[CopiesUpdate], streams: int, *,
+                       gather: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, want32: bool = False,
+                       store: bool = False):
+        """norm(sum_t gather[t] v_t) over the copies v of the stream with ``update`` in them (without ``gather`` their plain
+        sum); with ``store`` the v are kept.  ``x`` is [T, streams, width], or [T, width] while all copies are equal.
+        Returns (the stream, the rows in the model dtype, the rows in float32 if ``want32``)."""
+        from ..csrc import ops
+        count = rows.numel() if rows is not None else x.shape[0]
+        args = update.kernel_args(ctx) if update is not None else {}
+        kept = self.copies_buffer(ctx, x, streams) if store else None
+        summed = ctx.buffer("stream.copies_sum", (count, x.shape[-1]), torch.float32)
+        ops.stream_copies(x, streams, gather=gather, rows=rows, store=kept, out32=summed, **args)
+        act, act32 = self.forward(ctx, summed, want32=want32)
+        return x if kept is None else kept, act, act32
+
+    @staticmethod
+    def copies_buffer(ctx, x: torch.Tensor, streams: int) -> torch.Tensor:
+        """Where the copies are kept: x itself once it holds them, else a buffer beside the one row that stood for them."""
+        return x if x.dim() == 3 else ctx.buffer("stream.copies", (x.shape[0], streams, x.shape[-1]), torch.float32)
 
 
 class Position:
@@ -273,6 +322,10 @@ class Addition(Part):
         raise NotImplementedError
 
 
+class StreamConnection(Part):
+    """The constants with which a layer's sublayers read the copies of a stream and spread their outputs over them."""
+
+
 def shared_fetch(source: TensorSource, need: TensorNeed) -> torch.Tensor:
     """A tensor that several parts read (one table with a share per layer): fetched once per source and kept with it."""
     try:
@@ -293,6 +346,14 @@ class Block:
         # norms behind the sublayers, for the arrangements that have them
         self.mixer_out_norm, self.feed_forward_out_norm = mixer_out_norm, feed_forward_out_norm
         self.mixer_input: Optional[MixerInput] = None
+        self.connections: Optional[StreamConnection] = None
+
+    takes_connections: bool = False      # whether the arrangement runs on a stream that is kept as several copies
+
+    def set_connections(self, part: StreamConnection) -> None:
+        if not self.takes_connections:
+            raise ValueError(f"{type(self).__name__} runs on a single stream, not on copies of it")
+        self.connections = part
 
     takes_mixer_input: bool = False      # whether the arrangement has a place for a part in front of the mixer
 
@@ -303,7 +364,7 @@ class Block:
 
     def parts(self) -> list[Part]:
         """The block's parts; a layer without a feed-forward has neither it nor its norms."""
-        return [part for part in (self.mixer_norm, self.mixer_input, self.mixer, self.mixer_out_norm, self.feed_forward_norm,
+        return [part for part in (self.connections, self.mixer_norm, self.mixer_input, self.mixer, self.mixer_out_norm, self.feed_forward_norm,
                                   self.feed_forward, self.feed_forward_out_norm) if part is not None]
 
     def cache_need(self) -> CacheNeed:
@@ -322,7 +383,7 @@ class Block:
 
 _REGISTRIES: dict[str, dict[str, Callable[..., Any]]] = {
     "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "block": {}, "embedding": {}, "head": {},
-    "connector": {}, "addition": {}, "mixer_input": {},
+    "connector": {}, "addition": {}, "mixer_input": {}, "stream_connection": {},
 }
 
 

@@ -3,12 +3,12 @@
 left to the norm that follows it, which adds in float32 while it reads the stream.
 A second arrangement, ``output_norm``, has the norm behind the sublayer instead of in front of it; a third,
 ``parallel_pre_norm``, runs the two sublayers side by side on the same x; a fourth, ``sandwich_norm``, has a norm on
-both sides of each sublayer."""
+both sides of each sublayer; a fifth, ``hyper_connections``, is the first one on a stream that is kept as several copies."""
 from __future__ import annotations
 
 import torch
 
-from .base import Block, NormedUpdate, UpdateSum, as_tensor, register_part
+from .base import Block, CopiesUpdate, NormedUpdate, UpdateSum, as_tensor, register_part
 from .norm import LayerNorm
 
 
@@ -104,6 +104,30 @@ class SandwichNormBlock(Block):
         return x, NormedUpdate(self.feed_forward.forward_deferred(ctx, act2, act2_32), self.feed_forward_out_norm)
 
 
+class HyperConnectionBlock(Block):
+    """Pre-norm sublayers on a stream of several copies (``hyper_connections.py``): y = mixer(norm(sum_s in1[s] x_s)),
+    x_t <- sum_s mix1[s, t] x_s + out1[t] y, then the same for the feed-forward.  Between the two sublayers the copies
+    are not rewritten: the second norm reads what they would be, and the norm behind the layer stores them once, with both
+    sublayers' outputs and the product of the two mixes."""
+
+    takes_connections = True
+
+    def forward(self, ctx, x, pending, line, writes_cache):
+        c = self.connections
+        if c is None:
+            raise ValueError("a block on copies of the stream was given no connections")
+        x, act, _ = self.mixer_norm.forward_copies(ctx, x, pending, c.streams, gather=c.gather1, store=pending is not None)
+        y1 = as_tensor(ctx, self.mixer.forward(ctx, act, line, writes_cache))
+        if self.feed_forward is None:
+            return x, CopiesUpdate(c.mix1, first=y1, first_out=c.out1)
+        _, act2, act2_32 = self.feed_forward_norm.forward_copies(
+            ctx, x, CopiesUpdate(c.mix1, first=y1, first_out=c.out1), c.streams, gather=c.gather2,
+            want32=self.feed_forward.wants_float32_input)
+        y2 = self.feed_forward.forward_deferred(ctx, act2, act2_32)
+        return x, CopiesUpdate(c.mix_both, first=y1, first_out=c.out1_through, second=y2, second_out=c.out2)
+
+
+register_part("block", "hyper_connections", HyperConnectionBlock, replace=True)
 register_part("block", "sandwich_norm", SandwichNormBlock, replace=True)
 register_part("block", "parallel_pre_norm", ParallelPreNormBlock, replace=True)
 register_part("block", "pre_norm", PreNormBlock, replace=True)

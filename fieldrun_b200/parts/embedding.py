@@ -2,7 +2,7 @@
 and the vocabulary head: logits = rows @ W^T in float32, W the head's own matrix or the
 embedding's when tied (src/minimax.rs:54,373-376).  Two optional constants that the reference's
 model does not have: the embedding's ``scale`` (rows are multiplied by it) and the head's
-``softcap`` (logits <- cap * tanh(logits / cap)); ``typed_copy`` makes the embedding write the
+``scale`` (logits are multiplied by it) and ``softcap`` (then logits <- cap * tanh(logits / cap)); ``typed_copy`` makes the embedding write the
 stream a second time in the model dtype, for blocks whose sublayers read the stream itself.
 ``pair_table`` ``{"buckets", "mul_prev", "mul_cur"}`` adds a second row to every token's embedding, chosen by a hash
 of the token before and the token itself: row (previous * mul_prev + token * mul_cur) mod buckets of a table of
@@ -81,6 +81,7 @@ class VocabHead(Part):
         self.vocab_size = int(spec.args["vocab_size"])
         self.width = int(spec.args["width"])
         self.softcap = spec.args.get("softcap")
+        self.scale = float(spec.args.get("scale", 1.0))
         if self.softcap is not None and not float(self.softcap) > 0.0:
             raise ValueError(f"a logit cap of {self.softcap}")
         self.weight: Optional[torch.Tensor] = None
@@ -93,8 +94,8 @@ class VocabHead(Part):
 
     def forward(self, ctx, rows: torch.Tensor) -> torch.Tensor:
         logits = linear(rows, self.weight)
-        if self.softcap is not None:
-            ops.softcap(logits, float(self.softcap))
+        if self.softcap is not None or self.scale != 1.0:
+            ops.softcap(logits, self.softcap, self.scale)
         return logits
 
 

@@ -29,7 +29,7 @@ import torch
 from ..csrc import ops
 from ..weights.loader import MATRIX, VECTOR, TensorNeed, TensorSource
 from .base import FeedForward, UpdateSum, WeightedRows, register_part
-from .linear import linear
+from .linear import STREAM_ROWS, linear, one_tile
 
 TILE_ROWS = 32        # rows of one expert that a block of the expert kernels takes
 # Above this many rows per expert (on average) a step's expert products run on tcgen05: tiles of 32 rows and more
@@ -39,6 +39,30 @@ TILE_ROWS = 32        # rows of one expert that a block of the expert kernels ta
 # tokens crowd on fewer experts, and every tile beyond an expert's first reads its weights again (a prompt of 64
 # tokens: 525 against 419 us a layer, of 256: 1,400 against 617).
 TENSOR_CORE_ROWS_PER_EXPERT = {"decode": 4.0, "prompt": 1.0}
+
+
+FUSED_ACTIVATION_ROWS = 64      # from this many rows of a prompt step on, a dense unit's first product carries its activation
+
+
+class OneExpertTiles:
+    """The lists that make a step's rows one expert's rows in tiles, for the tcgen05 product; they depend on the number of
+    rows alone and are kept."""
+
+    def __init__(self):
+        self._made: dict = {}
+
+    def of(self, ctx, rows: int):
+        tile_rows = 256 if rows >= 256 else 128 if rows > 64 else 64 if rows > 32 else 32
+        key = (str(ctx.device), rows)
+        made = self._made.get(key)
+        if made is None:
+            if len(self._made) > 64:
+                self._made.clear()
+            count = (rows + tile_rows - 1) // tile_rows
+            flat = torch.tensor([0] * count + [tile_rows * i for i in range(count)] + [count, 0, rows], dtype=torch.int32).to(ctx.device)
+            made = self._made[key] = (flat[:count], flat[count:2 * count], flat[2 * count:2 * count + 1], flat[2 * count + 1:], count,
+                                      tile_rows)
+        return made
 
 
 class RoutedExperts(FeedForward):
@@ -88,7 +112,11 @@ class RoutedExperts(FeedForward):
         self._ones: Optional[torch.Tensor] = None
         if not 1 <= self.top_k <= self.num_experts:
             raise ValueError(f"top_k {self.top_k} is outside 1..{self.num_experts} experts")
-        if not (dtype == torch.bfloat16 and self.hidden_size % 128 == 0 and self.expert_width % 128 == 0):
+        # a shared expert without a gate per token is one expert whose rows are all rows: its first product carries its activation
+        self.shared_fused = bool(self.shared_width) and not self.shared_gate and dtype == torch.bfloat16
+        self.shared_tc = self.shared_fused and self.shared_width % 128 == 0 and self.hidden_size % 64 == 0
+        self.tiles = OneExpertTiles()
+        if not self.shared_tc and not (dtype == torch.bfloat16 and self.hidden_size % 128 == 0 and self.expert_width % 128 == 0):
             self.kernel_groups = ("common", "streams", "experts")      # sizes the tcgen05 products never take
         self.router: Optional[torch.Tensor] = None
         self.bias: Optional[torch.Tensor] = None
@@ -150,9 +178,21 @@ class RoutedExperts(FeedForward):
 
     def shared(self, ctx, act: torch.Tensor) -> torch.Tensor:
         """The shared expert's output [T, d] float32: silu(gate) * up, times the token's sigmoid gate where the part has one
-        (put on the hidden rows: the product behind it is linear), then the product out."""
+        (put on the hidden rows: the product behind it is linear), then the product out.  Without that gate a few rows' and a
+        prompt's first product carry the activation."""
+        rows = act.shape[0]
+        hidden = ctx.buffer("experts.shared_hidden", (rows, self.shared_width), self.dtype)
+        if self.shared_fused:
+            pair = self.w_shared_in[:2 * self.shared_width].view(1, 2 * self.shared_width, self.hidden_size)
+            if self.shared_tc and rows >= FUSED_ACTIVATION_ROWS and not ctx.is_decode:
+                tile_expert, tile_row0, num_tiles, offsets, count, tile_rows = self.tiles.of(ctx, rows)
+                ops.expert_gemm_tc(pair, act, tile_expert, tile_row0, num_tiles, offsets, count, tile_rows, hidden, paired=True)
+                return linear(hidden, self.w_shared_down)
+            if rows <= STREAM_ROWS and ops.weight_stream_takes(self.shared_width, self.hidden_size, paired=True):
+                tile_expert, tile_row0, num_tiles, offsets = one_tile(act.device, rows)
+                ops.weight_stream(pair, act, None, tile_expert, tile_row0, num_tiles, offsets, 1, 8, hidden, paired=True, lists_final=True)
+                return linear(hidden, self.w_shared_down)
         both = linear(act, self.w_shared_in)
-        hidden = ctx.buffer("experts.shared_hidden", (act.shape[0], self.shared_width), self.dtype)
         ops.gated_unit(both, hidden, "silu", row_gate=2 * self.shared_width if self.shared_gate else None)
         return linear(hidden, self.w_shared_down)
 
@@ -362,9 +402,6 @@ class DenseGatedUnit(FeedForward):
         return linear(hidden, self.w_down)
 
 
-FUSED_ACTIVATION_ROWS = 64      # from this many rows of a prompt step on, a dense unit's first product carries its activation
-
-
 class DenseUnit(FeedForward):
     """W_down act(W_up x): one product in, an activation, one product out.  ``activation`` is one of
     ``ops.ACTIVATIONS`` (``relu_squared``: relu(z)^2, ``gelu_tanh``, ``silu``, ``relu``).  A prompt's rows in bfloat16
@@ -392,7 +429,7 @@ class DenseUnit(FeedForward):
             self.kernel_groups = ("common", "streams")         # sizes the tcgen05 product never takes
         self.w_up: Optional[torch.Tensor] = None
         self.w_down: Optional[torch.Tensor] = None
-        self._tiles: dict = {}
+        self.tiles = OneExpertTiles()
 
     def _needs(self):
         d, i = self.hidden_size, self.width
@@ -409,21 +446,6 @@ class DenseUnit(FeedForward):
         self.w_up, self.w_down, *rest = (source.fetch(n) for n in self._needs())
         self.coefficients = rest[0] if rest else None
 
-    def fused_tiles(self, ctx, rows: int):
-        """The lists that make the step one expert's rows in tiles, for the tcgen05 product; they depend on the number
-        of rows alone and are kept."""
-        tile_rows = 256 if rows >= 256 else 128 if rows > 64 else 64 if rows > 32 else 32
-        key = (str(ctx.device), rows)
-        made = self._tiles.get(key)
-        if made is None:
-            if len(self._tiles) > 64:
-                self._tiles.clear()
-            count = (rows + tile_rows - 1) // tile_rows
-            flat = torch.tensor([0] * count + [tile_rows * i for i in range(count)] + [count, 0, rows], dtype=torch.int32).to(ctx.device)
-            made = self._tiles[key] = (flat[:count], flat[count:2 * count], flat[2 * count:2 * count + 1], flat[2 * count + 1:], count,
-                                       tile_rows)
-        return made
-
     def forward(self, ctx, act, act32):
         rows = act.shape[0]
         hidden = ctx.buffer("dense.hidden", (rows, self.width), self.dtype)
@@ -432,7 +454,7 @@ class DenseUnit(FeedForward):
         elif (self.dtype == torch.bfloat16 and rows >= FUSED_ACTIVATION_ROWS and not ctx.is_decode and self.width % 128 == 0
                 and self.hidden_size % 64 == 0):
             # a prompt's rows: product and activation in one kernel on tcgen05, the result rounded once to bfloat16
-            tile_expert, tile_row0, num_tiles, offsets, count, tile_rows = self.fused_tiles(ctx, rows)
+            tile_expert, tile_row0, num_tiles, offsets, count, tile_rows = self.tiles.of(ctx, rows)
             ops.expert_gemm_tc(self.w_up.view(1, self.width, self.hidden_size), act, tile_expert, tile_row0, num_tiles, offsets,
                                count, tile_rows, hidden, paired=False, activation=self.activation)
         else:

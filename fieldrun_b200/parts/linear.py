@@ -22,7 +22,7 @@ STREAM_ROWS = 8           # up to this many rows a dense product is a stream ove
 STREAM_FEATURES = 65536   # beyond this many output features the library product is at the memory roofline anyway
 
 
-def _one_tile(device: torch.device, rows: int):
+def one_tile(device: torch.device, rows: int):
     key = (str(device), rows)
     if key not in _ONE_TILE:
         zero = torch.zeros(1, dtype=torch.int32, device=device)
@@ -74,7 +74,7 @@ def linear(rows: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor]
         # few rows: the weight is the traffic; stream it once through the kernel that streams expert weights,
         # the dense layer being a single expert whose rows are all the rows
         tile_rows = 8 if count <= 8 else 16 if count <= 16 else 32
-        tile_expert, tile_row0, num_tiles, offsets = _one_tile(rows.device, count)
+        tile_expert, tile_row0, num_tiles, offsets = one_tile(rows.device, count)
         result = out if out is not None else torch.empty((count, features), dtype=torch.float32, device=rows.device)
         if ops.weight_stream_takes(features, inner, paired=False):
             # the lists of this one tile never change, so the weights may be on their way before the rows are ready

@@ -156,7 +156,7 @@ class DynamicTanh(Norm):
     """tanh(alpha v) * weight + bias with one learned scalar alpha: a norm without statistics.  Two of them that read
     the same stream (a block whose sublayers run side by side) go through one kernel (``forward_pair``), which also
     adds the updates that the block before left: float32 tensors and the experts' weighted rows.  ``forward_shifted``:
-    norm, updates and a token shift behind the norm in one pass."""
+    norm, updates and a token shift behind the norm in one pass; ``forward_copies``: the same for the copies of a stream."""
 
     replayable = True
     accepts_deferred = True
@@ -214,6 +214,18 @@ class DynamicTanh(Norm):
                 out32 = ctx.buffer(f"norm.out32.{self.width}", (count, self.width), torch.float32)
                 ops.dyt_norm(x, self.triple(), out32, rows=rows)       # x holds the sum by now (or nothing was added)
         return out, out32
+
+    def forward_copies(self, ctx, x, update, streams, *, gather=None, rows=None, want32=False, store=False):
+        """Update of the copies, their weighted sum and this norm of it in one pass."""
+        count = rows.numel() if rows is not None else x.shape[0]
+        out = ctx.buffer(f"norm.out.{self.width}", (count, self.width), self.dtype)
+        out32 = None
+        if want32 and self.dtype != torch.float32:
+            out32 = ctx.buffer(f"norm.out32.{self.width}", (count, self.width), torch.float32)
+        kept = self.copies_buffer(ctx, x, streams) if store else None
+        ops.stream_copies(x, streams, gather=gather, rows=rows, norm=self.triple(), store=kept, out=out, out32=out32,
+                          **(update.kernel_args(ctx) if update is not None else {}))
+        return x if kept is None else kept, out, (out if self.dtype == torch.float32 else out32) if want32 else None
 
     def forward_pair(self, ctx, x, other: "DynamicTanh", *, delta=None, want32=False):
         """This norm and ``other`` of the same x + delta (the sum stored back): (out, other's out, other's out in

@@ -119,6 +119,8 @@ class RandomInit:
             value = unit_normal(key, shape, device, self.norm_std)
         elif need.init == "around_half":                         # a positive scale well inside a tanh's bend
             value = unit_normal(key, shape, device, 0.5 * self.norm_std).add_(0.5)
+        elif need.init == "near_identity":                       # a square matrix that passes its input on, with some mixing
+            value = unit_normal(key, shape, device, self.norm_std) + torch.eye(shape[0], dtype=torch.float32, device=device)
         elif need.init == "bias":
             if self.bias_std == 0.0:
                 value = torch.zeros(shape, device=device, dtype=torch.float32)
