@@ -25,6 +25,9 @@ gated shared expert) beside a MiniMax-M2 model with as many experts of the same 
 turn, each behind a token shift; a feed-forward of normed powers) beside a Bamasun and a MiniMax-M2 model of equal width,
 projections and feed-forward weights.
 
+``--design kifunex``: a Kifunex model (four copies of the stream, windowed attention whose values are its keys, routed experts
+with a shared one) beside a MiniMax-M2 model with as many experts of the same size.
+
 The weights of every model are far larger than the L2 cache, and each timed step reads all of them.
 """
 from __future__ import annotations
@@ -164,6 +167,22 @@ def duzinex_config(width, heads, kv_heads, dim, ff, layers, vocab) -> dict[str, 
     return {"architecture": "Duzinex", "vocab": vocab, "width": width, "embedding": {"scale": 8.0}, "norm": {"eps": 1e-6}, "layers": listed}
 
 
+# the Kifunex comparison: experts as in the comparisons above plus a shared one, four copies of the stream
+KIFUNEX_EXPERTS, KIFUNEX_TOP, KIFUNEX_FF_SHARE, KIFUNEX_STREAMS, KIFUNEX_WINDOW = 16, 2, 4, 4, 1024
+
+
+def kifunex_config(width, heads, kv_heads, dim, ff, layers, vocab) -> dict[str, Any]:
+    """Every layer with tensors of its own: attention over a window whose values are its keys, routed experts and a shared
+    expert of an expert's size, on four copies of the stream."""
+    expert_ff = ff // KIFUNEX_FF_SHARE // 128 * 128
+    mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": KIFUNEX_EXPERTS, "top": KIFUNEX_TOP, "scale": 2.5},
+           "shared": {"ff": expert_ff}}
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": KIFUNEX_WINDOW},
+             "rot": {"base": 500000.0, "dims": dim // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    return {"architecture": "Kifunex", "vocab": vocab, "width": width, "streams": KIFUNEX_STREAMS, "norm": {"eps": 1e-6},
+            "logit_scale": 0.5, "logit_softcap": 30.0, "layers": [{"type": "attention", "mixer": mixer, "mlp": mlp} for _ in range(layers)]}
+
+
 def minimax_config(width, heads, kv_heads, dim, ff, layers, vocab, experts=None) -> dict[str, Any]:
     if experts is not None:
         count, top, expert_ff = experts
@@ -237,8 +256,13 @@ def _measure(lm, vocab: int, steps: int, warmup: int, decode_batches=(8, 64)) ->
             engine.record_steps = recording
         for s in slots:
             engine.release(s)
-    # ---- every kernel of one step of prompts
+    # ---- every kernel of one step of prompts (behind a step that brings back the buffers which the decode steps gave up)
     slots = [engine.new_sequence() for _ in range(PROMPTS_PER_STEP)]
+    engine.step(slots, prompts(PROMPTS_PER_STEP))
+    for s in slots:
+        engine.release(s)
+    slots = [engine.new_sequence() for _ in range(PROMPTS_PER_STEP)]
+    torch.cuda.synchronize()
     ops.timing_start()
     engine.step(slots, prompts(PROMPTS_PER_STEP))
     out["prefill_kernels_ms"] = {k: [n, round(v, 4)] for k, (n, v) in sorted(ops.timing_report().items())}
@@ -263,6 +287,9 @@ def compare_designs(sizes=("w2048", "w4096"), steps: int = 8, warmup: int = 3, d
         elif design == "depelix":
             experts = (DEPELIX_EXPERTS, DEPELIX_TOP, size["ff"] // DEPELIX_FF_SHARE // 128 * 128)
             pair = (("depelix", depelix_config(**size)), ("minimax_m2", minimax_config(**size, experts=experts)))
+        elif design == "kifunex":
+            experts = (KIFUNEX_EXPERTS, KIFUNEX_TOP, size["ff"] // KIFUNEX_FF_SHARE // 128 * 128)
+            pair = (("kifunex", kifunex_config(**size)), ("minimax_m2", minimax_config(**size, experts=experts)))
         elif design == "duzinex":
             pair = (("duzinex", duzinex_config(**size)), ("bamasun", bamasun_config(**size)), ("minimax_m2", minimax_config(**size)))
         else:

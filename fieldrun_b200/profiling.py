@@ -615,7 +615,32 @@ def attention_of_two_maps(kind: str, launches: int) -> dict:
     return {"case": f"maps_{kind}", "tokens": tokens, "ms": round(ms, 4), "tflops": round(2.0 * 2 * heads * seen * (dim + vdim) / ms / 1e9, 1)}
 
 
+def stream_copies(kind: str, launches: int, streams: int = 4) -> dict:
+    """The copies of a stream between two sublayers (stream_copies.cu), four copies of 2,048 columns, over 8,192 tokens or 64:
+    ``read`` behind a layer's mixer (the copies and one update read, two outputs), ``store`` behind a layer (the copies with two
+    updates, the second a shared expert's row and two experts' rows, read and stored, one output)."""
+    name, shape = kind.rsplit("_", 1)
+    tokens, width, top = 8192 if shape == "prefill" else 64, 2048, 2
+    x = torch.randn(tokens, streams, width, device=DEV)
+    y1, shared = torch.randn(tokens, width, device=DEV), torch.randn(tokens, width, device=DEV)
+    y, ew = torch.randn(tokens * top, width, device=DEV), torch.rand(tokens, top, device=DEV)
+    rowmap = torch.randperm(tokens * top, device=DEV).to(torch.int32)
+    ones = torch.ones(width, device=DEV)
+    mix, weights = torch.eye(streams, device=DEV) * 0.9, torch.full((streams,), 0.5, device=DEV)
+    out, out32 = torch.empty(tokens, width, dtype=torch.bfloat16, device=DEV), torch.empty(tokens, width, device=DEV)
+    common = dict(first=(y1, weights), mix=mix, gather=weights, norm=(ones, ones, ones[:1]), out=out)
+    if name == "read":
+        launch = lambda: ops.stream_copies(x, streams, out32=out32, **common)
+        floats = streams + 1 + 1
+    else:
+        launch = lambda: ops.stream_copies(x, streams, second=(shared,), experts=(y, ew, rowmap), second_out=weights, store=x, **common)
+        floats = 2 * streams + 2 + top
+    ms = _time(launch, launches) if shape == "prefill" else _time_recorded(launch, max(launches, 20))
+    return {"case": f"copies_{kind}", "tokens": tokens, "ms": round(ms, 4), "gbs": round(tokens * width * (4 * floats + 2) / ms / 1e6, 1)}
+
+
 CASES = {
+    **{f"copies_{kind}": (lambda n, kind=kind: stream_copies(kind, n)) for kind in ("read_prefill", "store_prefill", "read_decode", "store_decode")},
     **{f"maps_{kind}": (lambda n, kind=kind: attention_of_two_maps(kind, n))
        for kind in ("prefill", "prefill_plain", "prefill_two", "prefill_two_plain", "long", "long_plain", "long_two", "long_two_plain")},
     **{f"duzinex_{kind}": (lambda n, kind=kind: duzinex(kind, n))
