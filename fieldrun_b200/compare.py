@@ -250,6 +250,16 @@ def _measure(lm, vocab: int, steps: int, warmup: int, decode_batches=(8, 64)) ->
             # every kernel of one decode step, run directly
             recording, engine.record_steps = engine.record_steps, False
             engine.step(slots, [[1]] * batch)
+            routed = [block.feed_forward for block in lm.model.blocks if hasattr(block.feed_forward, "on_route")]
+            if routed:
+                # how many different experts a layer's weights are read of (tokens as the timed steps had them)
+                counts: list[int] = []
+                for part in routed:
+                    part.on_route = lambda ids: counts.append(len(torch.unique(ids)))
+                engine.step(slots, [[int(t)] for t in tokens])
+                for part in routed:
+                    part.on_route = None
+                out[f"decode_batch{batch}"]["experts_read_a_layer"] = round(sum(counts) / len(counts), 1)
             ops.timing_start()
             engine.step(slots, [[1]] * batch)
             out["decode_kernels_ms"] = {k: [n, round(v, 4)] for k, (n, v) in sorted(ops.timing_report().items())}
@@ -296,7 +306,9 @@ def compare_designs(sizes=("w2048", "w4096"), steps: int = 8, warmup: int = 3, d
             pair = (("bamasun", bamasun_config(**size)), ("minimax_m2", minimax_config(**size)))
         for design_name, config in pair:
             began = time.time()
-            lm = fr.random_model(config, fr.RandomInit(seed=1, matrix_std=0.02, norm_std=0.1, bias_std=0.02), dtype="bfloat16",
+            # dynamic-tanh norms give rows as small as the stream's: with biases beside them all tokens would pick the same experts
+            init = fr.RandomInit(seed=1, matrix_std=0.02, norm_std=0.1, bias_std=0.0 if design == "kifunex" else 0.02)
+            lm = fr.random_model(config, init, dtype="bfloat16",
                                  max_tokens=64 * (PROMPT + 256), num_slots=72, max_batch=64)
             entry[design_name] = _measure(lm, size["vocab"], steps, max(warmup, 3))
             entry[design_name]["build_s"] = round(time.time() - began, 1)

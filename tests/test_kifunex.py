@@ -115,7 +115,7 @@ def test_a_plan_with_copies_needs_connections_everywhere():
 
 @pytest.mark.parametrize("dims,base,blend", [
     (16, 1000.0, (8.0, 1.0, 4.0, 200.0)),            # all three ranges
-    (32, 10000.0, (4.0, 1.0, 4.0, 512.0 * 3)),
+    (32, 10000.0, (4.0, 1.0, 4.0, 1500.0)),
     (12, 20.0, (4.0, 1.0, 4.0, 1e6)),                # every wavelength stays
     (8, 300.0, (5.0, 1.0, 2.0, 3.0)),                # every wavelength is divided
     (2, 300.0, (5.0, 1.0, 1.0, 30.0)),               # nothing in between

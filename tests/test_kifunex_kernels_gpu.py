@@ -178,7 +178,7 @@ def test_a_norm_with_statistics_reads_copies_too(dtype):
 
 @BOTH
 @pytest.mark.parametrize("tokens", [5, 100])
-@pytest.mark.parametrize("heads,kv,dim,rot,biased", [(4, 2, 24, 16, False), (3, 3, 10, 10, True), (8, 1, 64, 32, False), (2, 1, 12, 0, True),
+@pytest.mark.parametrize("heads,kv,dim,rot,biased", [(4, 2, 24, 16, False), (3, 3, 10, 10, True), (5, 1, 64, 48, False), (2, 1, 12, 0, True),
                                                      (6, 2, 128, 128, False)])
 def test_values_are_the_keys_as_projected(dtype, tokens, heads, kv, dim, rot, biased):
     rng = np.random.default_rng(dim + tokens)
@@ -259,7 +259,7 @@ def test_window_in_the_general_kernel(dtype, heads, kv_heads, dim, window):
     close(f64(out), c["want"], KERNEL_TOL[dtype])
 
 
-TC_SIZES = [(8, 1, 64), (16, 1, 32), (6, 2, 128), (4, 4, 64), (12, 2, 96)]
+TC_SIZES = [(10, 1, 64), (16, 1, 32), (6, 2, 128), (4, 4, 64), (12, 2, 96)]
 
 
 @pytest.mark.parametrize("heads,kv_heads,dim", TC_SIZES)
@@ -369,7 +369,7 @@ def test_one_key_that_stands_out_at_a_windows_edge(dtype, heads, kv, dim, window
 # ------------------------------------------------------------------------------------------- experts and head
 
 @BOTH
-@pytest.mark.parametrize("hidden,experts,top,ff,shared,scale", [(96, 7, 3, 40, 56, 2.5), (42, 4, 4, 30, 22, 0.7), (128, 12, 2, 128, 256, 1.3),
+@pytest.mark.parametrize("hidden,experts,top,ff,shared,scale", [(96, 7, 3, 40, 56, 2.5), (42, 4, 4, 30, 22, 0.7), (128, 11, 3, 128, 256, 1.3),
                                                                 (256, 5, 1, 64, 128, 1.0), (64, 40, 6, 32, None, 1.7)])
 def test_experts_weighted_by_scores_without_renormalizing_and_a_shared_one(dtype, hidden, experts, top, ff, shared, scale):
     """Corrections large enough to change most choices; counts of rows that go through every routing and product kernel."""
@@ -410,7 +410,7 @@ def test_experts_weighted_by_scores_without_renormalizing_and_a_shared_one(dtype
 
 
 @BOTH
-@pytest.mark.parametrize("scale,cap", [(0.25, 15.0), (1.7, None), (1.0, 2.0), (1.0, None)])
+@pytest.mark.parametrize("scale,cap", [(0.3, 12.0), (1.7, None), (1.0, 2.0), (1.0, None)])
 def test_head_scales_then_caps(dtype, scale, cap):
     from test_parts_gpu import Stepper, lib, source
     _, config, _, parts, _ = lib()
